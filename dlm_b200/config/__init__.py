@@ -3,6 +3,8 @@ from .faguzen import FaguzenConfig
 from .qwen2_moe import Qwen2MoeConfig
 from .salolorn import SalolornConfig
 from .zasazen import ZasazenConfig
+from .zepilorn import ZepilornConfig
 from .zesapel import ZesapelConfig
 
-__all__ = ["ConfigError", "read_config_json", "FaguzenConfig", "Qwen2MoeConfig", "SalolornConfig", "ZasazenConfig", "ZesapelConfig"]
+__all__ = ["ConfigError", "read_config_json", "FaguzenConfig", "Qwen2MoeConfig", "SalolornConfig", "ZasazenConfig",
+           "ZepilornConfig", "ZesapelConfig"]

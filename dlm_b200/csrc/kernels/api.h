@@ -14,7 +14,8 @@ enum Epilogue : int {
     EPI_ADD = 1,      // out[m, n] += acc, out is float32 (the residual stream)
     EPI_SWIGLU = 2,   // out[m, n/2] = silu(acc[m, n]) * acc[m, n+1] for even n (interleaved weight rows)
     EPI_GELU = 3,     // out[m, n] = gelu(acc (+ bias[n])) in its exact (erf) form, stored as the output dtype
-    EPI_GELU_TANH = 4 // the same with gelu in its tanh form: z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))) / 2
+    EPI_GELU_TANH = 4,// the same with gelu in its tanh form: z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))) / 2
+    EPI_GEGLU_TANH = 5// EPI_SWIGLU with that gelu in place of silu
 };
 
 // out[T, H] (f32) = table[tokens[t], :] * scale
@@ -182,11 +183,11 @@ void gated_rmsnorm(const float* y, int ldy, const float* gate, int ldg, const fl
 // lddt); state f32 [slots, heads, N, P]; y f32 [T, heads * P].  Per head (group = head / (heads / groups)):
 // dt = softplus(dt_raw + dt_bias); S <- exp(-exp(A_log) dt) S + dt B x^T; y = S^T C + D x.
 // fixed_decay f32 [heads] != nullptr: S <- fixed_decay[head] S + B x^T instead (step size 1; dt_raw, dt_bias and
-// A_log are not read); D == nullptr: no direct term.  With groups == heads and rows [v | k | q] this is linear
+// A_log are not read); D == nullptr: no direct term.  silu_inputs != 0: x, B and C pass silu first.  With groups == heads and rows [v | k | q] this is linear
 // attention with a constant decay per head: S <- decay S + k v^T, y = S^T q.
 void ssm_scan(const float* xbc, int ldx, const float* dt_raw, int lddt, const float* dt_bias, const float* A_log,
               const float* D, float* state, const int32_t* cu_q, const int32_t* state_slot, float* y, int R, int heads,
-              int P, int N, int groups, const float* fixed_decay, cudaStream_t stream);
+              int P, int N, int groups, const float* fixed_decay, int silu_inputs, cudaStream_t stream);
 
 // Delta-rule scan.  proj f32 rows hold r, k, v and the raw removal rate at the given column offsets (heads * d
 // each); lw f32 [T, heads * d] the raw decay; state f32 [slots, heads, d, d] (key channel, value channel).
@@ -286,13 +287,15 @@ void gated_scan(const float* q, int ldq, const float* k, int ldk, const float* v
 // qkv f32 rows [q: nh * d | k: nkv * d | v: nkv * dv] (row stride ld).  Every q and k head is divided by its root
 // mean square over d (eps inside the root) and multiplied by qn_w / kn_w (f32 [d], shared by the heads; nullptr: that
 // side is not normed), then its first rot_dims entries are rotated by position * inv_freq[pair] (pair i is entries
-// (i, i + rot_dims / 2), or (2i, 2i + 1) with interleaved != 0).  q goes to q_out[T, nh * D] and, where slots !=
-// nullptr and slots[t] >= 0, k and v to the paged caches [pages, nkv, page_size, D], every head D wide with zeros
-// beyond its own size (D >= d, dv).
+// (i, i + rot_dims / 2), or (2i, 2i + 1) with interleaved != 0) with sines and cosines multiplied by `amplitude`.
+// norm_after != 0: the order is rotation, then division by the root mean square, and there are no weights.  q goes
+// to q_out[T, nh * D] and, where slots != nullptr and slots[t] >= 0, k and v to the paged caches [pages, nkv,
+// page_size, D], every head D wide with zeros beyond its own size (D >= d, dv).  slots == nullptr: only the query
+// heads are read.
 void head_norm_rope_write(const float* qkv, int ld, const int32_t* positions, const float* qn_w, const float* kn_w,
-                          float eps, const float* inv_freq, int rot_dims, int interleaved, const int32_t* slots,
-                          void* q_out, void* k_cache, void* v_cache, int T, int nh, int nkv, int d, int dv, int D,
-                          int page_size, int total_pages, int dtype, cudaStream_t stream);
+                          float eps, const float* inv_freq, int rot_dims, int interleaved, float amplitude, int norm_after,
+                          const int32_t* slots, void* q_out, void* k_cache, void* v_cache, int T, int nh, int nkv,
+                          int d, int dv, int D, int page_size, int total_pages, int dtype, cudaStream_t stream);
 
 // o[t, h * D + i] *= factor * sigmoid(gate[t * ldg + h]) in place (o in `dtype`, gate f32 raw)
 void head_gate(void* o, const float* gate, int ldg, int T, int nh, int D, float factor, int dtype, cudaStream_t stream);
@@ -333,5 +336,16 @@ void tanh_cap(float* x, long long n, float cap, cudaStream_t stream);
 // resid (f32 [T, W]) != nullptr: also resid[t, :] += bias[:]
 void entry_gate(void* o, const float* gate, int ldg, int T, int nh, int dv, int D, float factor, int dtype,
                 float* resid, const float* bias, int W, cudaStream_t stream);
+
+// ---- layers with a norm on their sublayers' outputs (postnorm.cu) ----
+
+// out[i] = norm(x[rows ? rows[i] : i]) with norm(v) = (v - mean) / sqrt(mean((v - mean)^2) + eps) * w + b  (x, w, b f32)
+void layer_norm(const float* x, const int32_t* rows, const float* w, const float* b, float eps, void* out, int n_rows,
+                int H, int out_dtype, cudaStream_t stream);
+// resid[t] += norm(y[t]) and, with out != nullptr, out[t] = the new resid[t] in out_dtype: a sublayer's closing norm,
+// the add and the next sublayer's input.  centered != 0: the norm above; 0: v / sqrt(mean(v^2) + eps) * w, without b
+// (nullptr).  clear != 0: y is left all zeros (for the next sublayer, which adds into it).
+void post_norm_add(float* resid, float* y, const float* w, const float* b, float eps, int centered, int clear, void* out,
+                   int T, int H, int out_dtype, cudaStream_t stream);
 
 }  // namespace dlmk

@@ -39,7 +39,7 @@ __device__ __forceinline__ float tanh_sfu(float x) {
 #endif
 
 // Which of the faster kernels take a chunked mask or a sink: the warp-level prefill kernel and every decode kernel
-// do; the tcgen05 prefill kernel does not (its steps go to the warp-level kernel then).
+// take both; the tcgen05 prefill kernel takes a sink but no chunks (its steps go to the warp-level kernel then).
 inline bool attention_prefill_takes(const Score&) { return true; }
 inline bool attention_decode_takes(const Score&, int /*dtype*/, int /*hd*/) { return true; }
 

@@ -47,6 +47,7 @@ struct PrefillTcParams {
     int R, nh, nkv, page_size, page_shift, total_pages, window;
     float scale_log2;
     float cap_in, cap_out;      // cap_out != 0: a score is cap_out * tanh(dot * cap_in), in base-2 units (a cap on the scores)
+    const float* sinks;         // f32 [nh] or nullptr: a logit per head in the softmax's denominator
     int skip_single;
     int* err;
 };
@@ -380,7 +381,14 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         }
         if (ok && __all_sync(0xffffffffu, mbar_wait(&pv_done[(n_tiles - 1) & 1], ((n_tiles - 1) >> 1) & 1, abort_flag))) {
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-            const float inv = l > 0.f ? 1.0f / l : 0.f;
+            float inv = l > 0.f ? 1.0f / l : 0.f;
+            if (p.sinks != nullptr && l > 0.f) {
+                // the sink (base-2 units) joins maximum and denominator: 2^m l / (2^m l + 2^sink)
+                const float sk = p.sinks[head] * 1.4426950408889634f;
+                const float top = fmaxf(m, sk);
+                const float a = ex2(m - top);
+                inv = a / (l * a + ex2(sk - top));
+            }
             const int Q = p.nh * HD;
             __nv_bfloat16* orow = p.out + (long long)(q_begin + q0 + row) * Q + head * HD;
 #pragma unroll 1
@@ -446,7 +454,7 @@ bool attention_prefill_tc_ok(const void* q, const void* k_cache, const void* v_c
                              int page_size, Score scale) {
     // (the row maximum is taken before the scores are scaled: the scale must be positive, and a distance term
     // has no place in that order of steps)
-    return scale.scale > 0.f && scale.slopes == nullptr && scale.plain_mask() && hd == HD && nkv > 0 && nh % nkv == 0 && page_size >= 64 && (page_size & (page_size - 1)) == 0 &&
+    return scale.scale > 0.f && scale.slopes == nullptr && scale.chunk <= 0 && hd == HD && nkv > 0 && nh % nkv == 0 && page_size >= 64 && (page_size & (page_size - 1)) == 0 &&
            ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k_cache) |
              reinterpret_cast<uintptr_t>(v_cache)) & 15) == 0;
 }
@@ -464,7 +472,7 @@ bool attention_prefill_tc(const void* q, const void* k_cache, const void* v_cach
     int shift = 0;
     while ((1 << shift) < page_size) ++shift;
     PrefillTcParams p{block_table, table_width, cu_q, kv_len, static_cast<__nv_bfloat16*>(out), R, nh, nkv, page_size,
-                      shift, total_pages, window, scale.scale * 1.4426950408889634f, scale.cap_in(), scale.cap_out(), skip_single,
+                      shift, total_pages, window, scale.scale * 1.4426950408889634f, scale.cap_in(), scale.cap_out(), scale.sinks, skip_single,
                       error_flag_ptr()};
     const size_t smem = (size_t)TILE_BYTES * 7 + 1024;      // Q, 2 x K, 2 x V, 2 x P, and room to align
     cudaFuncSetAttribute(attention_prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);

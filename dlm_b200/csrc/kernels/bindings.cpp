@@ -19,6 +19,7 @@ PYBIND11_MODULE(_dlm_kernels, m) {
     m.attr("EPI_SWIGLU") = (int)dlmk::EPI_SWIGLU;
     m.attr("EPI_GELU") = (int)dlmk::EPI_GELU;
     m.attr("EPI_GELU_TANH") = (int)dlmk::EPI_GELU_TANH;
+    m.attr("EPI_GEGLU_TANH") = (int)dlmk::EPI_GEGLU_TANH;
 
     m.def("embed", [](u64 tokens, u64 table, u64 out, int T, int H, int V, float scale, int dtype, u64 stream) {
         dlmk::embed(ptr<const int32_t>(tokens), ptr<const void>(table), ptr<float>(out), T, H, V, scale, dtype,
@@ -138,11 +139,11 @@ PYBIND11_MODULE(_dlm_kernels, m) {
     });
     m.def("ssm_scan", [](u64 xbc, int ldx, u64 dt_raw, int lddt, u64 dt_bias, u64 A_log, u64 D, u64 state, u64 cu_q,
                          u64 state_slot, u64 y, int R, int heads, int P, int N, int groups, u64 fixed_decay,
-                         u64 stream) {
+                         int silu_inputs, u64 stream) {
         dlmk::ssm_scan(ptr<const float>(xbc), ldx, ptr<const float>(dt_raw), lddt, ptr<const float>(dt_bias),
                        ptr<const float>(A_log), ptr<const float>(D), ptr<float>(state), ptr<const int32_t>(cu_q),
                        ptr<const int32_t>(state_slot), ptr<float>(y), R, heads, P, N, groups,
-                       ptr<const float>(fixed_decay), st(stream));
+                       ptr<const float>(fixed_decay), silu_inputs, st(stream));
     });
     m.def("delta_scan", [](u64 proj, int ld, int off_r, int off_k, int off_v, int off_a, u64 lw, int ldlw, u64 a_bias,
                            u64 state, u64 cu_q, u64 state_slot, u64 o, int R, int heads, int d, float unit_eps,
@@ -223,11 +224,12 @@ PYBIND11_MODULE(_dlm_kernels, m) {
                          q_scale, decay_kind, tau, st(stream));
     });
     m.def("head_norm_rope_write", [](u64 qkv, int ld, u64 positions, u64 qn_w, u64 kn_w, float eps, u64 inv_freq,
-                                     int rot_dims, int interleaved, u64 slots, u64 q_out, u64 k_cache, u64 v_cache, int T,
-                                     int nh, int nkv, int d, int dv, int D, int page_size, int total_pages, int dtype,
+                                     int rot_dims, int interleaved, float amplitude, int norm_after, u64 slots,
+                                     u64 q_out, u64 k_cache, u64 v_cache, int T, int nh, int nkv, int d, int dv, int D, int page_size, int total_pages, int dtype,
                                      u64 stream) {
         dlmk::head_norm_rope_write(ptr<const float>(qkv), ld, ptr<const int32_t>(positions), ptr<const float>(qn_w),
-                                   ptr<const float>(kn_w), eps, ptr<const float>(inv_freq), rot_dims, interleaved,
+                                   ptr<const float>(kn_w), eps, ptr<const float>(inv_freq), rot_dims, interleaved, amplitude,
+                                   norm_after,
                                    ptr<const int32_t>(slots), ptr<void>(q_out), ptr<void>(k_cache), ptr<void>(v_cache), T,
                                    nh, nkv, d, dv, D, page_size, total_pages, dtype, st(stream));
     });
@@ -268,6 +270,16 @@ PYBIND11_MODULE(_dlm_kernels, m) {
                            u64 bias, int W, u64 stream) {
         dlmk::entry_gate(ptr<void>(o), ptr<const float>(gate), ldg, T, nh, dv, D, factor, dtype, ptr<float>(resid),
                          ptr<const float>(bias), W, st(stream));
+    });
+    m.def("layer_norm", [](u64 x, u64 rows, u64 w, u64 b, float eps, u64 out, int n_rows, int H, int out_dtype,
+                           u64 stream) {
+        dlmk::layer_norm(ptr<const float>(x), ptr<const int32_t>(rows), ptr<const float>(w), ptr<const float>(b), eps,
+                         ptr<void>(out), n_rows, H, out_dtype, st(stream));
+    });
+    m.def("post_norm_add", [](u64 resid, u64 y, u64 w, u64 b, float eps, int centered, int clear, u64 out, int T, int H,
+                              int out_dtype, u64 stream) {
+        dlmk::post_norm_add(ptr<float>(resid), ptr<float>(y), ptr<const float>(w), ptr<const float>(b), eps, centered,
+                            clear, ptr<void>(out), T, H, out_dtype, st(stream));
     });
     m.def("take_error_flag", &dlmk::take_error_flag);
     m.def("reset_decode_merge_counters", [](u64 stream) { dlmk::reset_decode_merge_counters(st(stream)); });

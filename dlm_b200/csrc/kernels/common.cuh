@@ -107,5 +107,14 @@ __device__ __forceinline__ float gelu_tanh_f(float z) {
 template <int EPI> __device__ __forceinline__ float epi_act(float v) {
     return EPI == 3 ? gelu_exact_f(v) : (EPI == 4 ? gelu_tanh_f(v) : v);
 }
+// The gated epilogues, 2 (EPI_SWIGLU) and 5 (EPI_GEGLU_TANH): what the gate half goes through before it meets the up
+// half.  glu_act_fast: for results that are rounded to bfloat16 (fast exponential and division; the tanh form of gelu
+// is z times the logistic function of twice the tanh's argument).
+constexpr bool epi_is_glu(int epi) { return epi == 2 || epi == 5; }
+template <int EPI> __device__ __forceinline__ float glu_act(float g) { return EPI == 5 ? gelu_tanh_f(g) : silu_f(g); }
+template <int EPI> __device__ __forceinline__ float glu_act_fast(float g) {
+    const float z = EPI == 5 ? 1.59576912160573071176f * (g + 0.044715f * g * g * g) : g;
+    return __fdividef(g, 1.0f + __expf(-z));
+}
 
 }  // namespace dlmk

@@ -307,13 +307,15 @@ __global__ void gated_scan_kernel(const float* __restrict__ q, int ldq, const fl
 // ------------------------------------------------------------------- per-head norms, rotation, paged write
 // A warp a head: block (t, y) takes heads y * warps .. of token t.  x <- (x / sqrt(mean x^2 + eps)) * w over the
 // head's d entries (w shared by the heads; nullptr: no norm), kept in shared memory; then the first rot_dims entries
-// are rotated by position * inv_freq[pair], a lane a pair; q goes to q_out, k and v to the token's slot of the
-// paged caches, every head D wide with zeros beyond its own size.
-template <typename T>
+// are rotated by position * inv_freq[pair] with sines and cosines times `amplitude`, a lane a pair; q goes to q_out, k
+// and v to the token's slot of the paged caches, every head D wide with zeros beyond its own size.  AFTER: the heads
+// are rotated first and then divided by their root mean square, without weights (the rotated head stays in shared
+// memory until its sum is there).  Without slots only the query heads are read.
+template <typename T, bool AFTER>
 __global__ void head_norm_rope_write_kernel(const float* __restrict__ qkv, int ld, const int32_t* __restrict__ positions,
                                             const float* __restrict__ qn_w, const float* __restrict__ kn_w, float eps,
                                             const float* __restrict__ inv_freq, int rot_dims, int interleaved,
-                                            const int32_t* __restrict__ slots, T* __restrict__ q_out,
+                                            float amplitude, const int32_t* __restrict__ slots, T* __restrict__ q_out,
                                             T* __restrict__ k_cache, T* __restrict__ v_cache, int nh, int nkv, int d,
                                             int dv, int D, int page_size, int total_pages,
                                             int* err) {
@@ -332,9 +334,15 @@ __global__ void head_norm_rope_write_kernel(const float* __restrict__ qkv, int l
     }
     const long long page = slot >= 0 ? slot / page_size : 0, off = slot >= 0 ? slot % page_size : 0;
     float* sincos = head_stage + nwarp * d;                // [2][half]: the token's sines and cosines, once a block
-    for (int f = threadIdx.x; f < half; f += blockDim.x) sincosf(pos * inv_freq[f], sincos + f, sincos + half + f);
+    for (int f = threadIdx.x; f < half; f += blockDim.x) {
+        float sn, cs;
+        sincosf(pos * inv_freq[f], &sn, &cs);
+        sincos[f] = sn * amplitude;
+        sincos[half + f] = cs * amplitude;
+    }
     __syncthreads();
-    for (int hh = blockIdx.y * nwarp + warp; hh < nh + 2 * nkv; hh += gridDim.y * nwarp) {
+    const int n_heads = slots != nullptr ? nh + 2 * nkv : nh;
+    for (int hh = blockIdx.y * nwarp + warp; hh < n_heads; hh += gridDim.y * nwarp) {
         if (hh >= nh + nkv) {                               // a value head: copied as it is
             if (slot < 0) continue;
             const int g = hh - nh - nkv;
@@ -354,7 +362,7 @@ __global__ void head_norm_rope_write_kernel(const float* __restrict__ qkv, int l
             sh[i] = x;
             ss = fmaf(x, x, ss);
         }
-        if (w != nullptr) {
+        if (!AFTER && w != nullptr) {
             ss = warp_sum(ss);
             const float inv = 1.0f / sqrtf(ss / (float)d + eps);
             for (int i = lane; i < d; i += 32) sh[i] = (sh[i] * inv) * w[i];      // a lane rereads what it wrote
@@ -362,6 +370,26 @@ __global__ void head_norm_rope_write_kernel(const float* __restrict__ qkv, int l
         __syncwarp();
         T* dst = is_q ? q_out + ((long long)t * nh + hh) * D
                       : k_cache + ((page * nkv + (hh - nh)) * page_size + off) * D;
+        if (AFTER) {
+            ss = 0.f;
+            for (int f = lane; f < half; f += 32) {         // a lane a pair, in place
+                const int ia = interleaved ? 2 * f : f, ib = interleaved ? 2 * f + 1 : f + half;
+                const float x = sh[ia], y = sh[ib];
+                const float sn = sincos[f], cs = sincos[half + f];
+                const float a = x * cs - y * sn, b = y * cs + x * sn;
+                sh[ia] = a;
+                sh[ib] = b;
+                ss = fmaf(a, a, ss);
+                ss = fmaf(b, b, ss);
+            }
+            for (int i = 2 * half + lane; i < d; i += 32) ss = fmaf(sh[i], sh[i], ss);
+            ss = warp_sum(ss);
+            const float inv = 1.0f / sqrtf(ss / (float)d + eps);
+            __syncwarp();
+            for (int i = lane; i < D; i += 32) dst[i] = from_f32<T>(i < d ? sh[i] * inv : 0.f);
+            __syncwarp();
+            continue;
+        }
         for (int f = lane; f < half; f += 32) {             // a lane a pair
             const int ia = interleaved ? 2 * f : f, ib = interleaved ? 2 * f + 1 : f + half;
             const float x = sh[ia], y = sh[ib];
@@ -575,29 +603,34 @@ void memory_scan(const float* q, int ldq, const float* k, int ldk, const float* 
 }
 
 void head_norm_rope_write(const float* qkv, int ld, const int32_t* positions, const float* qn_w, const float* kn_w,
-                          float eps, const float* inv_freq, int rot_dims, int interleaved, const int32_t* slots,
-                          void* q_out, void* k_cache, void* v_cache, int T, int nh, int nkv, int d, int dv, int D,
-                          int page_size, int total_pages, int dtype, cudaStream_t stream) {
+                          float eps, const float* inv_freq, int rot_dims, int interleaved, float amplitude, int norm_after,
+                          const int32_t* slots, void* q_out, void* k_cache, void* v_cache, int T, int nh, int nkv,
+                          int d, int dv, int D, int page_size, int total_pages, int dtype, cudaStream_t stream) {
     if (T <= 0) return;
     DLM_CHECK(D >= d && D >= dv, "head_norm_rope_write: the stored head size must hold keys and values");
     DLM_CHECK(rot_dims % 2 == 0 && rot_dims >= 0 && rot_dims <= d, "head_norm_rope_write: rotated dims must be even and <= d");
     DLM_CHECK(rot_dims == 0 || inv_freq != nullptr, "head_norm_rope_write: a rotation needs its table");
     int* err = error_flag_ptr();
     const int warps = 8;
-    int gy = (nh + 2 * nkv + warps - 1) / warps;            // a head a warp while the blocks are few (a decode step);
+    const int n_heads = slots != nullptr ? nh + 2 * nkv : nh;
+    DLM_CHECK(!norm_after || (qn_w == nullptr && kn_w == nullptr), "head_norm_rope_write: a norm after the rotation has no weights");
+    int gy = (n_heads + warps - 1) / warps;            // a head a warp while the blocks are few (a decode step);
     while (gy > 1 && (long long)T * gy > 16 * 148) gy = (gy + 1) / 2;   // on a prompt several heads a warp: a block's
     const dim3 grid(T, gy);                                  // opening (slot, sines) is most of a one-head warp's work
     const size_t stage = ((size_t)warps * d + rot_dims) * sizeof(float);
     DLM_CHECK(stage <= 48 * 1024, "head_norm_rope_write: head size too large");
-    if (dtype == F32)
-        launch_dep(head_norm_rope_write_kernel<float>, grid, dim3(32 * warps), stage, stream, qkv, ld, positions, qn_w, kn_w, eps,
-                   inv_freq, rot_dims, interleaved, slots, static_cast<float*>(q_out), static_cast<float*>(k_cache),
-                   static_cast<float*>(v_cache), nh, nkv, d, dv, D, page_size, total_pages, err);
-    else
-        launch_dep(head_norm_rope_write_kernel<__nv_bfloat16>, grid, dim3(32 * warps), stage, stream, qkv, ld, positions, qn_w,
-                   kn_w, eps, inv_freq, rot_dims, interleaved, slots, static_cast<__nv_bfloat16*>(q_out),
-                   static_cast<__nv_bfloat16*>(k_cache), static_cast<__nv_bfloat16*>(v_cache), nh, nkv, d, dv, D,
-                   page_size, total_pages, err);
+#define DLM_HNRW(T, AFTER)                                                                                           \
+    launch_dep(head_norm_rope_write_kernel<T, AFTER>, grid, dim3(32 * warps), stage, stream, qkv, ld, positions, qn_w,   \
+               kn_w, eps, inv_freq, rot_dims, interleaved, amplitude, slots, static_cast<T*>(q_out),                     \
+               static_cast<T*>(k_cache), static_cast<T*>(v_cache), nh, nkv, d, dv, D, page_size, total_pages, err)
+    if (dtype == F32) {
+        if (norm_after) DLM_HNRW(float, true);
+        else DLM_HNRW(float, false);
+    } else {
+        if (norm_after) DLM_HNRW(__nv_bfloat16, true);
+        else DLM_HNRW(__nv_bfloat16, false);
+    }
+#undef DLM_HNRW
     check_launch("head_norm_rope_write");
 }
 

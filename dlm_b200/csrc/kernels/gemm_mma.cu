@@ -165,9 +165,9 @@ __global__ void __launch_bounds__(THREADS) gemm_mma_kernel(MmaParams p) {
             for (int j = 0; j < NTW; ++j) {
                 const int col = n0 + wn * 32 + j * 8 + 2 * t;
                 const float v0 = acc[i][j][half * 2], v1 = acc[i][j][half * 2 + 1];
-                if (EPI == EPI_SWIGLU) {
+                if (epi_is_glu(EPI)) {
                     if (col + 1 < p.N)
-                        static_cast<TOut*>(p.out)[(long long)row * p.ldo + (col >> 1)] = from_f32<TOut>(silu_f(v0) * v1);
+                        static_cast<TOut*>(p.out)[(long long)row * p.ldo + (col >> 1)] = from_f32<TOut>(glu_act<EPI>(v0) * v1);
                 } else if (EPI == EPI_ADD) {
                     float* o = static_cast<float*>(p.out) + (long long)row * p.ldo;
                     if (col < p.N) o[col] += v0;
@@ -195,6 +195,7 @@ void launch_bm(const MmaParams& p, int epilogue, dim3 grid, cudaStream_t stream)
         case EPI_ADD: DLM_MMA(EPI_ADD, float) break;
         case EPI_GELU: DLM_MMA(EPI_GELU, TOut) break;
         case EPI_GELU_TANH: DLM_MMA(EPI_GELU_TANH, TOut) break;
+        case EPI_GEGLU_TANH: DLM_MMA(EPI_GEGLU_TANH, TOut) break;
         default: DLM_MMA(EPI_SWIGLU, TOut) break;
     }
 #undef DLM_MMA
@@ -206,7 +207,7 @@ void gemm_mma(const void* a, int lda, const int32_t* a_rows, const void* w, int 
               const int32_t* expert_offsets, int num_experts, const float* bias, void* out, int ldo, int M, int N,
               int K, int out_dtype, int epilogue, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return;
-    DLM_CHECK(epilogue != EPI_SWIGLU || N % 2 == 0, "gemm: the SwiGLU epilogue needs an even N");
+    DLM_CHECK(!epi_is_glu(epilogue) || N % 2 == 0, "gemm: a gated epilogue needs an even N");
     DLM_CHECK(epilogue != EPI_ADD || out_dtype == F32, "gemm: the accumulate epilogue needs a float32 output");
     DLM_CHECK(bias == nullptr || epilogue == EPI_STORE || epilogue == EPI_GELU || epilogue == EPI_GELU_TANH, "gemm: a bias goes with a storing epilogue only");
     MmaParams p{static_cast<const __nv_bfloat16*>(a), lda, a_rows, static_cast<const __nv_bfloat16*>(w), ldw,

@@ -173,7 +173,7 @@ __global__ void __launch_bounds__(WARPS * 32) gemm_smallm_kernel(SmallParams p) 
         __syncthreads();
 
         const int m_here = min(MP, m_count - m0);
-        if (EPI == EPI_SWIGLU) {
+        if (epi_is_glu(EPI)) {
             // element = (tile r', row of A, pair of weight rows)
             for (int i = tid; i < R * MP * 8; i += WARPS * 32) {
                 const int pr = i & 7, m = (i >> 3) % MP, rr = i / (8 * MP);
@@ -185,7 +185,7 @@ __global__ void __launch_bounds__(WARPS * 32) gemm_smallm_kernel(SmallParams p) 
                     up += red[rr * S + ss][2 * pr + 1][m];
                 }
                 static_cast<TOut*>(p.out)[(long long)(row0 + m0 + m) * p.ldo + (n >> 1)] =
-                    from_f32<TOut>(silu_f(gate) * up);
+                    from_f32<TOut>(glu_act<EPI>(gate) * up);
             }
         } else {
             for (int i = tid; i < R * MP * 16; i += WARPS * 32) {
@@ -209,6 +209,7 @@ void launch_nt(const SmallParams& p, int epilogue, dim3 grid, cudaStream_t strea
         case EPI_ADD: launch_dep(gemm_smallm_kernel<NT, EPI_ADD, float>, grid, WARPS * 32, 0, stream, p); break;
         case EPI_GELU: launch_dep(gemm_smallm_kernel<NT, EPI_GELU, TOut>, grid, WARPS * 32, 0, stream, p); break;
         case EPI_GELU_TANH: launch_dep(gemm_smallm_kernel<NT, EPI_GELU_TANH, TOut>, grid, WARPS * 32, 0, stream, p); break;
+        case EPI_GEGLU_TANH: launch_dep(gemm_smallm_kernel<NT, EPI_GEGLU_TANH, TOut>, grid, WARPS * 32, 0, stream, p); break;
         default: launch_dep(gemm_smallm_kernel<NT, EPI_SWIGLU, TOut>, grid, WARPS * 32, 0, stream, p); break;
     }
 }
@@ -226,7 +227,7 @@ void gemm_smallm(const void* a, int lda, const int32_t* a_rows, const void* w, i
                  const int32_t* expert_offsets, int num_experts, const float* bias, void* out, int ldo, int M, int N,
                  int K, int out_dtype, int epilogue, int rows_per_pass, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return;
-    DLM_CHECK(epilogue != EPI_SWIGLU || N % 2 == 0, "gemm: the SwiGLU epilogue needs an even N");
+    DLM_CHECK(!epi_is_glu(epilogue) || N % 2 == 0, "gemm: a gated epilogue needs an even N");
     DLM_CHECK(epilogue != EPI_ADD || out_dtype == F32, "gemm: the accumulate epilogue needs a float32 output");
     SmallParams p;
     p.a = static_cast<const __nv_bfloat16*>(a); p.lda = lda; p.a_rows = a_rows;

@@ -343,7 +343,7 @@ __global__ void __launch_bounds__(THREADS, 1) gemm_stream_kernel(StreamParams p)
                 const int out_row0 = wk.row0 + pass * MP, m_here = min(MP, wk.m_count - pass * MP), n_base = wk.tile * RT;
                 if (!mbar_wait(&red_full[e & 1], (e >> 1) & 1, abort_flag)) { ok = false; break; }
                 const float* rb = red + (size_t)(e & 1) * CW * 16 * (MP + 1);
-                if (EPI == EPI_SWIGLU) {
+                if (epi_is_glu(EPI)) {
                     // element = (row of A, pair of weight rows)
 #pragma unroll
                     for (int i = lane; i < MP * 8; i += 32) {
@@ -357,7 +357,7 @@ __global__ void __launch_bounds__(THREADS, 1) gemm_stream_kernel(StreamParams p)
                             up += rb[((size_t)ww * 16 + 2 * pr + 1) * (MP + 1) + m];
                         }
                         static_cast<TOut*>(p.out)[(long long)(out_row0 + m) * p.ldo + (n >> 1)] =
-                            from_f32<TOut>(silu_f(gate) * up);
+                            from_f32<TOut>(glu_act<EPI>(gate) * up);
                     }
                 } else {
 #pragma unroll
@@ -401,6 +401,8 @@ void launch_nt(const StreamParams& p, int grid, int out_dtype, int epilogue, cud
                        else launch_one<NT, NCH, EPI_GELU, __nv_bfloat16>(p, grid, stream); break;
         case EPI_GELU_TANH: if (f32) launch_one<NT, NCH, EPI_GELU_TANH, float>(p, grid, stream);
                        else launch_one<NT, NCH, EPI_GELU_TANH, __nv_bfloat16>(p, grid, stream); break;
+        case EPI_GEGLU_TANH: if (f32) launch_one<NT, NCH, EPI_GEGLU_TANH, float>(p, grid, stream);
+                       else launch_one<NT, NCH, EPI_GEGLU_TANH, __nv_bfloat16>(p, grid, stream); break;
         default: if (f32) launch_one<NT, NCH, EPI_SWIGLU, float>(p, grid, stream);
                  else launch_one<NT, NCH, EPI_SWIGLU, __nv_bfloat16>(p, grid, stream); break;
     }
@@ -432,7 +434,7 @@ void gemm_stream(const void* a, int lda, const int32_t* a_rows, const void* w, i
                  const int32_t* expert_offsets, int num_experts, const float* bias, void* out, int ldo, int M, int N,
                  int K, int out_dtype, int epilogue, int rows_per_pass, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return;
-    DLM_CHECK(epilogue != EPI_SWIGLU || N % 2 == 0, "gemm: the SwiGLU epilogue needs an even N");
+    DLM_CHECK(!epi_is_glu(epilogue) || N % 2 == 0, "gemm: a gated epilogue needs an even N");
     DLM_CHECK(epilogue != EPI_ADD || out_dtype == F32, "gemm: the accumulate epilogue needs a float32 output");
     StreamParams p;
     p.a = static_cast<const __nv_bfloat16*>(a); p.lda = lda; p.a_rows = a_rows;

@@ -250,7 +250,7 @@ bool gemm_tc(const void* a, int lda, const void* w, int ldw, const int32_t* expe
              const float* bias, void* out, int ldo, int M, int N, int K, int out_dtype, int epilogue,
              cudaStream_t stream) {
     if (M <= 0 || N <= 0) return true;
-    DLM_CHECK(epilogue != EPI_SWIGLU || N % 2 == 0, "gemm: the SwiGLU epilogue needs an even N");
+    DLM_CHECK(!epi_is_glu(epilogue) || N % 2 == 0, "gemm: a gated epilogue needs an even N");
     DLM_CHECK(epilogue != EPI_ADD || out_dtype == F32, "gemm: the accumulate epilogue needs a float32 output");
     DLM_CHECK(bias == nullptr || epilogue == EPI_STORE || epilogue == EPI_GELU || epilogue == EPI_GELU_TANH, "gemm: a bias goes with a storing epilogue only");
     if (N > BM && gemm_tc_pair_enabled() &&
@@ -286,6 +286,8 @@ bool gemm_tc(const void* a, int lda, const void* w, int ldw, const int32_t* expe
                        else launch<G, EPI_GELU, __nv_bfloat16>(mw, ma, p, nx, total_tiles, stream); break;  \
         case EPI_GELU_TANH: if (f32) launch<G, EPI_GELU_TANH, float>(mw, ma, p, nx, total_tiles, stream);        \
                        else launch<G, EPI_GELU_TANH, __nv_bfloat16>(mw, ma, p, nx, total_tiles, stream); break;  \
+        case EPI_GEGLU_TANH: if (f32) launch<G, EPI_GEGLU_TANH, float>(mw, ma, p, nx, total_tiles, stream);      \
+                       else launch<G, EPI_GEGLU_TANH, __nv_bfloat16>(mw, ma, p, nx, total_tiles, stream); break; \
         default: if (f32) launch<G, EPI_SWIGLU, float>(mw, ma, p, nx, total_tiles, stream);                 \
                  else launch<G, EPI_SWIGLU, __nv_bfloat16>(mw, ma, p, nx, total_tiles, stream); break;      \
     }

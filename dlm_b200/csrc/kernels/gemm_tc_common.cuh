@@ -74,7 +74,7 @@ __device__ __forceinline__ void epilogue_tile(const TcParams& p, float* st, uint
         const int tok0 = row_begin + c0;
         const int n_valid = min(CH, row_end - tok0);      // tokens of this chunk that exist
         if (n_valid <= 0) continue;                       // uniform over the warp
-        if (EPI == EPI_SWIGLU) {
+        if (epi_is_glu(EPI)) {
             // Even lanes hold gate, their odd neighbours up, for the same output.  Per pair of tokens (j, j + 1)
             // the two lanes swap one number: the even lane sends its gate of token j + 1 and gets the up of
             // token j, so the even lane finishes token j and the odd lane token j + 1: one exchange and one
@@ -86,7 +86,7 @@ __device__ __forceinline__ void epilogue_tile(const TcParams& p, float* st, uint
                 const float a0 = __uint_as_float(v[j]), a1 = __uint_as_float(v[j + 1]);
                 const float got = __shfl_xor_sync(0xffffffffu, odd ? a0 : a1, 1);
                 const float g = odd ? got : a0, uu = odd ? a1 : got;
-                st[(j + (odd ? 1 : 0)) * 17 + (lane >> 1)] = __fdividef(g, 1.0f + __expf(-g)) * uu;
+                st[(j + (odd ? 1 : 0)) * 17 + (lane >> 1)] = glu_act_fast<EPI>(g) * uu;
             }
             __syncwarp();
             TOut* o = static_cast<TOut*>(p.out) + (long long)tok0 * p.ldo + (colw >> 1);

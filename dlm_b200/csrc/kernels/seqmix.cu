@@ -329,7 +329,7 @@ __global__ void ssm_scan_kernel(const float* __restrict__ xbc, int ldx, const fl
                                 const float* __restrict__ dt_bias, const float* __restrict__ A_log,
                                 const float* __restrict__ D, float* state, const int32_t* __restrict__ cu_q,
                                 const int32_t* __restrict__ state_slot, float* y, int heads, int P, int N, int groups,
-                                int parts, int tile, int wide, const float* __restrict__ fixed_decay) {
+                                int parts, int tile, int wide, const float* __restrict__ fixed_decay, int silu_inputs) {
     dep_wait();          // nothing is read or written before the kernels before this one have ended
     // (a long kernel, launched in the ordinary way: its blocks are placed when the machine is free, and the
     // kernel after it is let in only when it ends)
@@ -400,6 +400,13 @@ __global__ void ssm_scan_kernel(const float* __restrict__ xbc, int ldx, const fl
             const float dt = fixed ? 1.0f : softplus_f(row[2 * N + cols] + bias);
             row[2 * N + cols] = dt;
             row[2 * N + cols + 1] = fixed ? decay_h : expf(a * dt);
+        }
+        if (silu_inputs) {                   // B, C and x lie side by side in a token's row
+            const int w = 2 * N + min(cols, P - p0);
+            for (int idx = threadIdx.x; idx < n * w; idx += blockDim.x) {
+                float* v = buf + (size_t)(idx / w) * rl + idx % w;
+                *v = silu_f(*v);
+            }
         }
         __syncthreads();
         // (unrolled: a token depends on the one before it through the state's own multiply-add only, so the sums
@@ -758,7 +765,7 @@ void gated_rmsnorm(const float* y, int ldy, const float* gate, int ldg, const fl
 
 void ssm_scan(const float* xbc, int ldx, const float* dt_raw, int lddt, const float* dt_bias, const float* A_log,
               const float* D, float* state, const int32_t* cu_q, const int32_t* state_slot, float* y, int R, int heads,
-              int P, int N, int groups, const float* fixed_decay, cudaStream_t stream) {
+              int P, int N, int groups, const float* fixed_decay, int silu_inputs, cudaStream_t stream) {
     if (R <= 0) return;
     DLM_CHECK(fixed_decay != nullptr || (dt_raw != nullptr && dt_bias != nullptr && A_log != nullptr && D != nullptr),
               "ssm_scan: without fixed decays the step sizes, their bias, A_log and D are needed");
@@ -785,7 +792,7 @@ void ssm_scan(const float* xbc, int ldx, const float* dt_raw, int lddt, const fl
             cudaFuncSetAttribute(ssm_scan_kernel<NPT, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);    \
         ssm_scan_kernel<NPT, V><<<grid, cols * parts, smem, stream>>>(xbc, ldx, dt_raw, lddt, dt_bias, A_log, D, state, \
                                                                      cu_q, state_slot, y, heads, P, N, groups, parts, \
-                                                                     tile, wide, fixed_decay);                        \
+                                                                     tile, wide, fixed_decay, silu_inputs);           \
     } while (0)
     if (vec) {
         if (per <= 4) DLM_SSM(4, true);

@@ -215,10 +215,18 @@ class NativeOps:
                              _p(row_scale), self._stream())
         return out
 
-    def ssm_scan(self, xbc, dt_raw, dt_bias, A_log, D, state, batch, heads, P, N, groups, fixed_decay=None):
+    def ssm_scan(self, xbc, dt_raw, dt_bias, A_log, D, state, batch, heads, P, N, groups, fixed_decay=None,
+                 silu_inputs=False):
         """State-space scan over each request's tokens; ``state`` ``[slots, heads, N, P]`` is read and left
-        up to date.  Returns y ``[T, heads * P]`` in 32-bit."""
+        up to date.  Returns y ``[T, heads * P]`` in 32-bit.  ``silu_inputs``: x, B and C pass silu first (``xbc``
+        may or may not hold the result afterwards)."""
         T = xbc.shape[0]
+        if silu_inputs and T > 64:
+            # on a prompt one pass over the rows is cheaper than every block of the scan doing its own
+            self.launches += 1
+            self.k.activation(_p(xbc), xbc.stride(0), _p(xbc), xbc.stride(0), T, xbc.shape[1], self._ACTS["silu"], _F32,
+                              self._stream())
+            silu_inputs = False
         assert xbc.shape[1] == heads * P + 2 * groups * N and xbc.dtype == torch.float32 and xbc.stride(1) == 1
         assert state.shape[1:] == (heads, N, P)
         assert fixed_decay is not None or (dt_raw.shape == (T, heads) and dt_raw.stride(1) == 1)
@@ -226,7 +234,7 @@ class NativeOps:
         self.launches += 1
         self.k.ssm_scan(_p(xbc), xbc.stride(0), _p(dt_raw), 0 if dt_raw is None else dt_raw.stride(0), _p(dt_bias),
                         _p(A_log), _p(D), _p(state), _p(batch.cu_q), _p(batch.state_slot), _p(y), batch.num_requests,
-                        heads, P, N, groups, _p(fixed_decay), self._stream())
+                        heads, P, N, groups, _p(fixed_decay), int(bool(silu_inputs)), self._stream())
         return y
 
     def delta_scan(self, proj, offsets, lw, a_bias, state, batch, heads, d, unit_eps, decay_coef):
@@ -367,19 +375,22 @@ class NativeOps:
         return o
 
     def head_norm_rope_write(self, qkv, positions, qn_w, kn_w, eps, inv_freq, rot_dims, interleaved, slots, k_cache,
-                             v_cache, nh, nkv, d, dv, D, out_dtype):
+                             v_cache, nh, nkv, d, dv, D, out_dtype, amplitude=1.0, norm_after=False):
         """RMS norm of every query and key head over its ``d`` entries (weights ``[d]`` shared by the heads; None: no
         norm), rotary positions on the first ``rot_dims`` entries, q returned ``[T, nh * D]`` and k, v written at the
-        tokens' slots, every head ``D`` wide (zeros beyond its own size)."""
+        tokens' slots, every head ``D`` wide (zeros beyond its own size).  ``amplitude``: a factor on sines and cosines.
+        ``norm_after``: the heads are rotated first and then divided by their root mean square (no weights).
+        ``slots`` None: only the query heads are read and nothing is written."""
         T = qkv.shape[0]
-        assert qkv.dtype == torch.float32 and qkv.stride(1) == 1 and qkv.shape[1] >= (nh + nkv) * d + nkv * dv
+        assert qkv.dtype == torch.float32 and qkv.stride(1) == 1
+        assert qkv.shape[1] >= (nh * d if slots is None else (nh + nkv) * d + nkv * dv)
         total_pages, nkv_c, page_size, D_c = k_cache.shape
         assert (nkv_c, D_c) == (nkv, D) and k_cache.dtype == out_dtype and v_cache.shape == k_cache.shape
         q = torch.empty((T, nh * D), dtype=out_dtype, device=qkv.device)
         self.launches += 1
         self.k.head_norm_rope_write(_p(qkv), qkv.stride(0), _p(positions), _p(qn_w), _p(kn_w), float(eps), _p(inv_freq),
-                                    int(rot_dims), int(bool(interleaved)), _p(slots), _p(q), _p(k_cache), _p(v_cache), T,
-                                    nh, nkv, d, dv, D, page_size, total_pages, _dt(out_dtype), self._stream())
+                                    int(rot_dims), int(bool(interleaved)), float(amplitude), int(bool(norm_after)),
+                                    _p(slots), _p(q), _p(k_cache), _p(v_cache), T, nh, nkv, d, dv, D, page_size, total_pages, _dt(out_dtype), self._stream())
         return q
 
     def head_gate(self, o, gate, nh, D, factor=1.0):
@@ -407,6 +418,31 @@ class NativeOps:
         assert x0 is None or (x0.shape == (T, H) and x0.is_contiguous() and x0.dtype == torch.float32)
         self.launches += 1
         self.k.add_vec_rows(_p(x), _p(x0), _p(vec), T, H, self._stream())
+
+    # ------------------------------------- norms on sublayers' outputs
+    def layer_norm(self, x, w, b, eps, out_dtype, rows=None):
+        """``(x - mean) / sqrt(mean((x - mean)^2) + eps) * w + b`` of the 32-bit rows x (only ``rows`` of them when
+        given) in ``out_dtype``."""
+        H = x.shape[-1]
+        assert x.dtype == torch.float32 and x.is_contiguous() and w.shape == (H,) and b.shape == (H,)
+        n = x.shape[0] if rows is None else rows.numel()
+        out = torch.empty((n, H), dtype=out_dtype, device=x.device)
+        self.launches += 1
+        self.k.layer_norm(_p(x), _p(rows), _p(w), _p(b), float(eps), _p(out), n, H, _dt(out_dtype), self._stream())
+        return out
+
+    def post_norm_add(self, resid, y, w, b, eps, out_dtype, clear=False):
+        """``resid += norm(y)``; the norm is centred with weight and bias, or (``b`` None) an RMS norm with a weight.
+        Returns the new residual in ``out_dtype`` (``resid`` itself when that is 32-bit).  ``clear``: y is left all
+        zeros."""
+        T, H = resid.shape
+        assert resid.dtype == torch.float32 and resid.is_contiguous() and y.shape == (T, H) and y.is_contiguous()
+        assert y.dtype == torch.float32 and w.shape == (H,) and (b is None or b.shape == (H,))
+        out = None if out_dtype == torch.float32 else torch.empty((T, H), dtype=out_dtype, device=resid.device)
+        self.launches += 1
+        self.k.post_norm_add(_p(resid), _p(y), _p(w), _p(b), float(eps), int(b is not None), int(bool(clear)), _p(out),
+                             T, H, _dt(out_dtype), self._stream())
+        return resid if out is None else out
 
     # ------------------------------------- squashing norms and caps, a gate per entry, the max-gated matrix memory
     def dyt_norm(self, x, w, b, alpha, out_dtype, rows=None):
@@ -561,9 +597,16 @@ class NativeOps:
         return self.activation(self.linear(a, w, None, torch.float32), act, a.dtype)
 
     def linear_swiglu(self, a, w_gate_up):
+        return self.linear_glu(a, w_gate_up, "silu")
+
+    def linear_glu(self, a, w_gate_up, act):
+        """``act(gate) * up`` of a product with interleaved gate and up rows, as an epilogue; ``act`` "silu" or
+        "gelu_tanh"."""
         (M, K), N = a.shape, w_gate_up.shape[0]
+        assert w_gate_up.shape[1] == K and a.dtype == w_gate_up.dtype
         out = torch.empty((M, N // 2), dtype=a.dtype, device=a.device)
-        self._gemm(a, w_gate_up, out, M, N, K, self.k.EPI_SWIGLU)
+        epi = {"silu": self.k.EPI_SWIGLU, "gelu_tanh": self.k.EPI_GEGLU_TANH}[act]
+        self._gemm(a, w_gate_up, out, M, N, K, epi)
         return out
 
     def grouped_swiglu(self, a, w_gate_up, offsets, rows):

@@ -30,6 +30,8 @@ class GroupedQueryAttention(Mixer):
         self.qkv_bias = qkv_bias          # None: decided by the presence of the bias tensors
         self.window = int(window) if window else None
         self.position = build_part("position", position) if position is not None else None
+        if self.position is not None and self.position.amplitude != 1.0:
+            raise ValueError("this mixer's kernel takes no factor on sines and cosines")
         self.q_dim, self.kv_dim = self.nh * self.hd, self.nkv * self.hd
         self.scale = 1.0 / math.sqrt(self.hd)
         self.w_qkv = self.b_qkv = self.w_o = None
@@ -276,10 +278,14 @@ class HeadNormedAttention(Mixer):
     A query at p sees key ``j <= p`` iff ``p - j < window`` (when a window is given) and
     ``floor(j / chunk) == floor(p / chunk)`` (when a chunk size is given; chunks are counted from position 0 of the
     request).  With ``sink`` the softmax's denominator also holds ``exp(sink_n)``, a learned logit per head that has
-    no key and no value and is not scaled.  ``gate`` True or ``"head"``: head n's output is multiplied by
+    no key and no value and is not scaled; ``sink_logit`` instead gives a logit that is a constant.  ``gate`` True or ``"head"``: head n's output is multiplied by
     ``sigmoid(W_g h)_n`` (``g`` is ``[heads, hidden]``); ``"entry"``: the heads side by side are multiplied entry by
     entry by ``sigmoid(W_g h)`` (``g`` is ``[heads * vdim, hidden]``).  The gate reads the same input as the
     projections.  The output is ``out_scale * (W_o [heads side by side] + o.b)`` (the bias with ``o_bias``).
+
+    ``qk_norm="after"``: the heads are rotated first, then divided by their root mean square, and there are no norm
+    weights.  ``own_kv`` False: the layer has no key and value projections (nor their norms and biases) and its call
+    reads the cache of an earlier call, with the queries, mask, scale, sink and gate of its own.
 
     Keys and values are cached with one head size (the larger of ``dim`` and ``vdim``, rounded up to a size the
     tensor-core kernels take; zeros beyond a head's own, zero columns in ``W_o``).  A chunked mask never looks back
@@ -289,16 +295,23 @@ class HeadNormedAttention(Mixer):
     _HEAD_SIZES = (16, 32, 48, 64, 96, 128)
 
     def __init__(self, hidden_size: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, eps: float,
-                 qk_norm: bool = True, position: PartSpec | None = None, window: int | None = None,
+                 qk_norm: bool | str = True, position: PartSpec | None = None, window: int | None = None,
                  chunk: int | None = None, sink: bool = False, gate: bool | str = False, out_scale: float = 1.0,
-                 qkv_bias: bool = False, o_bias: bool = False, softcap: float | None = None):
+                 qkv_bias: bool = False, o_bias: bool = False, softcap: float | None = None,
+                 sink_logit: float | None = None, own_kv: bool = True):
         if heads % kv_heads:
             raise ValueError("heads must be a multiple of kv_heads")
         if gate not in (False, True, "head", "entry"):
             raise ValueError(f"gate must be False, True, 'head' or 'entry', got {gate!r}")
+        if qk_norm not in (False, True, "after"):
+            raise ValueError(f"qk_norm must be False, True or 'after', got {qk_norm!r}")
+        if sink and sink_logit is not None:
+            raise ValueError("the sink's logit is either learned or a constant")
+        self.sink_logit = None if sink_logit is None else float(sink_logit)
+        self.own_kv, self.norm_after = bool(own_kv), qk_norm == "after"
         self.hidden, self.H, self.G, self.d, self.dv = int(hidden_size), int(heads), int(kv_heads), int(dim), int(vdim)
         self.scale, self.eps, self.out_scale = float(scale), float(eps), float(out_scale)
-        self.qk_norm, self.has_sink, self.has_gate = bool(qk_norm), bool(sink), bool(gate)
+        self.qk_norm, self.has_sink, self.has_gate = qk_norm is True, bool(sink), bool(gate)
         self.gate_rows = self.H * self.dv if gate == "entry" else self.H          # rows of W_g
         self.qkv_bias, self.o_bias = bool(qkv_bias), bool(o_bias)
         self.softcap = float(softcap) if softcap else 0.0
@@ -311,15 +324,14 @@ class HeadNormedAttention(Mixer):
 
     def param_specs(self):
         H, G, d, dv = self.H, self.G, self.d, self.dv
-        specs = [ParamSpec("q", (H * d, self.hidden)), ParamSpec("k", (G * d, self.hidden)),
-                 ParamSpec("v", (G * dv, self.hidden)), ParamSpec("o", (self.hidden, H * dv))]
+        rows = {"q": H * d, "k": G * d, "v": G * dv} if self.own_kv else {"q": H * d}
+        specs = [ParamSpec(n, (r, self.hidden)) for n, r in rows.items()] + [ParamSpec("o", (self.hidden, H * dv))]
         if self.qkv_bias:
-            specs += [ParamSpec("q.b", (H * d,), init="bias"), ParamSpec("k.b", (G * d,), init="bias"),
-                      ParamSpec("v.b", (G * dv,), init="bias")]
+            specs += [ParamSpec(n + ".b", (r,), init="bias") for n, r in rows.items()]
         if self.o_bias:
             specs.append(ParamSpec("o.b", (self.hidden,), init="bias"))
         if self.qk_norm:
-            specs += [ParamSpec("q.norm", (d,), init="norm"), ParamSpec("k.norm", (d,), init="norm")]
+            specs += [ParamSpec(n + ".norm", (d,), init="norm") for n in ("q", "k") if n in rows]
         if self.has_sink:
             specs.append(ParamSpec("sink", (H,), init="bias"))
         if self.has_gate:
@@ -327,10 +339,10 @@ class HeadNormedAttention(Mixer):
         return specs
 
     def load(self, tensors, rt: Runtime):
-        names = ("q", "k", "v", "g") if self.has_gate else ("q", "k", "v")
-        self.w_in = torch.cat([rt.matrix(tensors[n]) for n in names], dim=0).contiguous()
+        names = ["q", "k", "v"] if self.own_kv else ["q"]
+        self.w_in = torch.cat([rt.matrix(tensors[n]) for n in names + ["g"] * self.has_gate], dim=0).contiguous()
         if self.qkv_bias:       # the gate has no bias: zeros for its rows
-            parts = [rt.vector(tensors[n + ".b"]) for n in "qkv"]
+            parts = [rt.vector(tensors[n + ".b"]) for n in names]
             if self.has_gate:
                 parts.append(torch.zeros(self.gate_rows, dtype=torch.float32, device=rt.device))
             self.b_in = torch.cat(parts).contiguous()
@@ -344,8 +356,11 @@ class HeadNormedAttention(Mixer):
         self.w_o = rt.matrix(w_o)
         self.b_o = (rt.vector(tensors["o.b"]) * self.out_scale).contiguous() if self.o_bias else None
         if self.qk_norm:
-            self.qn, self.kn = rt.vector(tensors["q.norm"]), rt.vector(tensors["k.norm"])
+            self.qn = rt.vector(tensors["q.norm"])
+            self.kn = rt.vector(tensors["k.norm"]) if self.own_kv else None
         self.sink = rt.vector(tensors["sink"]) if self.has_sink else None
+        if self.sink_logit is not None:
+            self.sink = torch.full((self.H,), self.sink_logit, dtype=torch.float32, device=rt.device)
         if self.position is not None:
             self.position.rotary(rt)        # the table is made now: no copy from the host in the middle of a step
 
@@ -361,20 +376,23 @@ class HeadNormedAttention(Mixer):
         rt, ops, b = ctx.rt, ctx.rt.ops, ctx.batch
         H, G, d, dv = self.H, self.G, self.d, self.dv
         view = ctx.paged(call)
+        if view.write and not self.own_kv:
+            raise RuntimeError(f"layer call {call} has no key and value projections and reads no other call's cache")
         proj = ops.linear(h, self.w_in, self.b_in, torch.float32)          # [q | k | v | gate]
         rot = self.position.rotary(rt) if self.position is not None else None
         inv_freq, rot_dims = rot if rot is not None else (None, 0)
         q = ops.head_norm_rope_write(proj, b.positions, self.qn, self.kn, self.eps, inv_freq, rot_dims,
                                      bool(rot is not None and self.position.interleaved),
                                      view.group.slots if view.write else None, view.k, view.v, H, G, d, dv, self.D,
-                                     rt.dtype)
+                                     rt.dtype, amplitude=self.position.amplitude if rot is not None else 1.0,
+                                     norm_after=self.norm_after)
         extra = {"softcap": self.softcap} if self.softcap else {}
         o = ops.attention(q, view.k, view.v, view.group.block_table, b.cu_q, b.kv_len, self.window or 0, self.scale,
                           H, G, self.D, b.max_q_len, b.max_kv_len, b.num_single, chunk=self.chunk or 0, sinks=self.sink,
                           **extra)
         bias = self.b_o                                # the output bias still to be added (None: none, or done)
         if self.has_gate:
-            g = proj[:, (H + G) * d + G * dv:]
+            g = proj[:, (H * d + (G * (d + dv) if self.own_kv else 0)):]
             if self.gate_rows == H:
                 ops.head_gate(o, g, H, self.D, self.out_scale)
             else:

@@ -141,14 +141,26 @@ class Norm(Part):
         32-bit result."""
         return None
 
+    def closing(self) -> "tuple[torch.Tensor, torch.Tensor | None, float] | None":
+        """``(weight, bias, eps)`` if a kernel may apply this norm to a sublayer's output itself while it adds it to the
+        residual: with a bias the centred norm, with bias None the plain RMS norm.  None: the caller asks ``forward``."""
+        rms = self.fusable_rms()
+        return None if rms is None else (rms[0], None, rms[1])
+
+    def scale_output(self, factor: torch.Tensor) -> None:
+        """Multiplies the norm's output entry by entry by ``factor`` (32-bit, once, after ``load``): a learned scale
+        behind a norm joins the norm's own weights."""
+        raise NotImplementedError(f"{type(self).__name__} cannot take a factor on its output")
+
 
 class PositionEncoding(Part):
     """``rotary()`` returns None or ``(inv_freq f32[rotary_dim/2] on the device, rotary_dim)``:
     pair i of each head is rotated by ``position * inv_freq[i]``; dimensions from ``rotary_dim``
     on pass through.  Pair i is dims ``(i, i + rotary_dim/2)``, or ``(2i, 2i + 1)`` when the
-    class attribute ``interleaved`` is True."""
+    class attribute ``interleaved`` is True.  Sines and cosines are multiplied by ``amplitude``."""
 
     interleaved = False
+    amplitude = 1.0
 
     def rotary(self, rt: Runtime):
         return None
@@ -231,6 +243,8 @@ class StepContext:
         self.batch = batch
         self._paged = paged_of_call
         self._state = state_of_call
+        self._rounded = None        # (call, rows): what ``leave_rounded`` was given last
+        self._zeroed = None         # rows of zeros that a block is done with
 
     def paged(self, call: int) -> PagedView:
         v = self._paged(call)
@@ -245,3 +259,26 @@ class StepContext:
         if s is None:
             raise RuntimeError(f"layer call {call} asked for per-request state {name!r} but declared no need for it")
         return s
+
+    # ---- rows that blocks with a norm on their sublayers' outputs hand on to each other within a step
+    def rounded(self, call: int, resid: torch.Tensor) -> torch.Tensor:
+        """The residual in the activation dtype: what the block of the call before left, else a copy made now (in
+        32-bit the residual itself)."""
+        if self.rt.dtype == torch.float32:
+            return resid
+        if self._rounded is not None and self._rounded[0] == call - 1:
+            return self._rounded[1]
+        return self.rt.ops.activation(resid, "copy", self.rt.dtype)
+
+    def leave_rounded(self, call: int, rows: "torch.Tensor | None") -> None:
+        """``rows``: the residual after ``call``, rounded (None: whoever changes the residual without rounding it)."""
+        self._rounded = None if rows is None else (call, rows)
+
+    def take_zeroed(self, like: torch.Tensor) -> torch.Tensor:
+        """32-bit rows of zeros of ``like``'s shape for a sublayer to add into; ``give_zeroed`` takes them back once
+        they are zeros again."""
+        z, self._zeroed = self._zeroed, None
+        return z if z is not None and z.shape == like.shape else torch.zeros_like(like)
+
+    def give_zeroed(self, rows: torch.Tensor) -> None:
+        self._zeroed = rows

@@ -141,6 +141,60 @@ class SandwichBlock(ParallelBlock):
         self._close(resid, y, self.norm2b, None, rt)
 
 
+class PostNormBlock(ParallelBlock):
+    """Norms on the sublayers' outputs only: ``x += s1 * norm1(mixer(x))``, then ``x += s2 * norm2(ffn(x))``; the sublayers
+    read x itself.  ``layer_scale``: the learned scales ``s1`` and ``s2`` (``[hidden_size]``) exist; they join the norms'
+    weights at load.  ``ffn`` None: only the first sublayer.
+
+    A sublayer adds its output into rows of zeros.  Where the norm lets a kernel apply it (``Norm.closing``), the norm,
+    the add to the residual, the next sublayer's rounded input and the clearing of those rows are one pass, and the
+    rows serve every sublayer of the step."""
+
+    def __init__(self, norm1: PartSpec, mixer: PartSpec, norm2: PartSpec | None = None, ffn: PartSpec | None = None,
+                 hidden_size: int | None = None, layer_scale: bool = False, names: dict[str, str] | None = None):
+        super().__init__(norm1, mixer, norm2, ffn, names={"scale1": "scale1", "scale2": "scale2", **(names or {})})
+        if layer_scale and hidden_size is None:
+            raise ValueError("a layer scale needs hidden_size")
+        self.hidden = hidden_size
+        self.layer_scale = bool(layer_scale)
+
+    def _scales(self):
+        if not self.layer_scale:
+            return []
+        out = [(self.names["scale1"], self.norm1)]
+        return out + [(self.names["scale2"], self.norm2)] if self.ffn is not None else out
+
+    def param_specs(self):
+        return super().param_specs() + [ParamSpec(n, (int(self.hidden),), init="norm") for n, _ in self._scales()]
+
+    def load(self, tensors, rt):
+        super().load(tensors, rt)
+        for name, norm in self._scales():
+            norm.scale_output(rt.vector(tensors[name]))
+
+    @staticmethod
+    def _close(resid, y, norm, rt):
+        """``resid += norm(y)``, y zeroed; the new residual in the activation dtype."""
+        fused = norm.closing()
+        if fused is not None:
+            return rt.ops.post_norm_add(resid, y, *fused, rt.dtype, clear=True)
+        resid += norm.forward(y, rt, out_dtype=torch.float32)
+        y.zero_()
+        return resid if rt.dtype == torch.float32 else rt.ops.activation(resid, "copy", rt.dtype)
+
+    def forward(self, resid, ctx: StepContext, call: int):
+        rt = ctx.rt
+        h = ctx.rounded(call, resid)
+        y = ctx.take_zeroed(resid)
+        self.mixer.forward(h, y, ctx, call)
+        h = self._close(resid, y, self.norm1, rt)
+        if self.ffn is not None:
+            self.ffn.forward(h, y, ctx, pre_norm=None)
+            h = self._close(resid, y, self.norm2, rt)
+        ctx.give_zeroed(y)
+        ctx.leave_rounded(call, h)
+
+
 class HyperConnectionBlock(Part):
     """A pre-norm layer over S residual streams ``xs[:, s]`` instead of one.  For sublayer q (1: the mixer,
     2: the feed-forward) with learned ``in_q[S]``, ``mix_q[S, S]`` (indexed [from, to]) and ``out_q[S]``::
@@ -253,4 +307,5 @@ class HyperConnectionBlock(Part):
 register_part("block", "prenorm", PreNormBlock)
 register_part("block", "parallel", ParallelBlock)
 register_part("block", "sandwich", SandwichBlock)
+register_part("block", "postnorm", PostNormBlock)
 register_part("block", "hyper_connections", HyperConnectionBlock)

@@ -17,10 +17,15 @@ def interleave_gate_up(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
 
 
 class DenseSwiGLU(FeedForward):
-    """``resid += down · (silu(gate·h) ⊙ up·h)`` without biases (src/forward/cpu.rs:966-971, 1198)."""
+    """``resid += down · (act(gate·h) ⊙ up·h)`` without biases (src/forward/cpu.rs:966-971, 1198); ``activation`` "silu"
+    or "gelu_tanh" (gelu in its tanh form), either in the first product's epilogue."""
 
-    def __init__(self, hidden_size: int, intermediate_size: int, names: dict[str, str] | None = None):
+    def __init__(self, hidden_size: int, intermediate_size: int, names: dict[str, str] | None = None,
+                 activation: str = "silu"):
         """``names``: the three tensors' names, by default the ones of Qwen2-MoE checkpoints."""
+        if activation not in ("silu", "gelu_tanh"):
+            raise ValueError(f"unknown activation {activation!r}")
+        self.act = activation
         self.hidden, self.inter = int(hidden_size), int(intermediate_size)
         self.names = {"gate": "gate_proj.weight", "up": "up_proj.weight", "down": "down_proj.weight"}
         if names:
@@ -39,7 +44,7 @@ class DenseSwiGLU(FeedForward):
 
     def forward(self, h, resid, ctx: StepContext, pre_norm=None):
         ops = ctx.rt.ops
-        act = ops.linear_swiglu(h, self.w_gate_up)
+        act = ops.linear_glu(h, self.w_gate_up, self.act)
         ops.linear_add(act, self.w_down, resid)
 
 

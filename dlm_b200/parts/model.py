@@ -151,7 +151,8 @@ class DecoderModel:
 
     # --------------------------------------------------------------- cache
     def cache_needs(self):
-        """Per call of the order: (PagedCache or None, RequestState or None, owner call index)."""
+        """Per call of the order: (PagedCache or None, RequestState or None, owner call index).  A cache that other
+        calls read keeps what the furthest-looking of them (and of its owner) needs."""
         out = []
         for ci, c in enumerate(self.order):
             block = self.blocks[c.layer]
@@ -159,6 +160,10 @@ class DecoderModel:
             # a block with state of its own (beside its mixer's) says so itself
             state = block.state_need() if hasattr(block, "state_need") else block.mixer.state_need()
             out.append((block.mixer.cache_need(), state, owner))
+        for ci, (need, _, owner) in enumerate(out):
+            own = out[owner][0]
+            if owner != ci and own.window is not None and (need.window is None or need.window > own.window):
+                out[owner] = (replace(own, window=need.window), *out[owner][1:])
         return out
 
     # ---------------------------------------------------------------- step
@@ -189,6 +194,7 @@ class DecoderModel:
         for ci, c in enumerate(self.order):
             if c.enters_pass is not None:
                 x = self.pass_entry.forward(x, x0, c.enters_pass, rt)
+                ctx.leave_rounded(ci, None)
             self.blocks[c.layer].forward(x, ctx, ci)
             if self.after_layer is not None:
                 self.after_layer(ci, x)

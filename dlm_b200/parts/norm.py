@@ -32,6 +32,33 @@ class RMSNorm(Norm):
     def fusable_rms(self):
         return self.weight, self.eps
 
+    def scale_output(self, factor):
+        self.weight = (self.weight * factor).contiguous()
+
+
+class LayerNorm(Norm):
+    """``(x - mean) / sqrt(mean((x - mean)^2) + eps) * weight + bias``, all of it 32-bit, the result stored in the
+    activation dtype.  Tensors: the weight (``param``) and ``<param>.b``."""
+
+    def __init__(self, size: int, eps: float, param: str = "weight"):
+        self.size, self.eps, self.param = int(size), float(eps), str(param)
+        self.weight = self.bias = None
+
+    def param_specs(self):
+        return [ParamSpec(self.param, (self.size,), init="norm"), ParamSpec(self.param + ".b", (self.size,), init="bias")]
+
+    def load(self, tensors, rt: Runtime):
+        self.weight, self.bias = rt.vector(tensors[self.param]), rt.vector(tensors[self.param + ".b"])
+
+    def forward(self, x, rt: Runtime, rows=None, out_dtype=None):
+        return rt.ops.layer_norm(x, self.weight, self.bias, self.eps, out_dtype or rt.dtype, rows)
+
+    def closing(self):
+        return self.weight, self.bias, self.eps
+
+    def scale_output(self, factor):
+        self.weight, self.bias = (self.weight * factor).contiguous(), (self.bias * factor).contiguous()
+
 
 class DynamicTanh(Norm):
     """A norm that takes no statistics: ``out = tanh(alpha * x) * weight + bias`` entry by entry, with one learned
@@ -65,4 +92,5 @@ class DynamicTanh(Norm):
 
 
 register_part("norm", "rmsnorm", RMSNorm)
+register_part("norm", "layernorm", LayerNorm)
 register_part("norm", "dynamic_tanh", DynamicTanh)

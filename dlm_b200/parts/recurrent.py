@@ -185,10 +185,20 @@ class RetentionMixer(Mixer):
 
     Each head's o is divided by its root mean square (no weight), the heads side by side are multiplied by
     ``silu(W_g h)``, then ``W_o``.  The scan is the state-space scan with constant decays and step size 1 (keys as
-    its B, queries as its C, one group per head)."""
+    its B, queries as its C, one group per head).
+
+    ``activation="silu"``: q, k and v pass silu (there is then no rotation).  ``key_scale``: another factor on k.
+    ``norm="all"``: the heads side by side are normed together instead of each by itself; ``norm_weight``: the norm has
+    a weight (``norm``, ``[heads * vdim]``).  ``gate``: "silu" or "sigmoid"."""
 
     def __init__(self, hidden_size: int, heads: int, dim: int, vdim: int, decay: list[float], eps: float,
-                 rope_base: float | None = None, rope_dims: int = 0):
+                 rope_base: float | None = None, rope_dims: int = 0, activation: str | None = None,
+                 key_scale: float | None = None, norm: str = "head", norm_weight: bool = False, gate: str = "silu"):
+        if activation not in (None, "silu") or norm not in ("head", "all") or gate not in ("silu", "sigmoid"):
+            raise ValueError(f"unknown activation {activation!r}, norm {norm!r} or gate {gate!r}")
+        self.silu, self.norm_all, self.has_norm_w, self.gate = activation == "silu", norm == "all", bool(norm_weight), gate
+        self.key_scale = float(dim) ** -0.5 if key_scale is None else float(key_scale)
+        self.norm_w = None
         self.hidden, self.H, self.d, self.dv, self.eps = int(hidden_size), int(heads), int(dim), int(vdim), float(eps)
         self.decay = [float(v) for v in decay]
         if len(self.decay) != self.H:
@@ -197,19 +207,24 @@ class RetentionMixer(Mixer):
         self.rope_base = float(rope_base) if rope_base is not None else 0.0
         if self.rope_dims % 2 or not (0 <= self.rope_dims <= self.d):
             raise ValueError(f"rope_dims must be even and at most dim, got {self.rope_dims}")
+        self.turns = self.rope_dims > 0 or self.key_scale != 1.0        # a pass over q and k before the scan
+        if self.silu and self.turns:
+            raise ValueError("activated queries and keys take neither a rotation nor a factor")
         self.w_in = self.w_o = self._freq = self._decay = None
 
     def param_specs(self):
         H, d, dv = self.H, self.d, self.dv
         return [ParamSpec("q", (H * d, self.hidden)), ParamSpec("k", (H * d, self.hidden)),
                 ParamSpec("v", (H * dv, self.hidden)), ParamSpec("g", (H * dv, self.hidden)),
-                ParamSpec("o", (self.hidden, H * dv))]
+                ParamSpec("o", (self.hidden, H * dv))] + \
+            ([ParamSpec("norm", (H * dv,), init="norm")] if self.has_norm_w else [])
 
     def load(self, tensors, rt: Runtime):
         # rows [v | k | q | g]: the scan reads values, keys and queries side by side in that order
         self.w_in = torch.cat([rt.matrix(tensors[n]) for n in ("v", "k", "q", "g")], dim=0).contiguous()
         self.w_o = rt.matrix(tensors["o"])
         self._decay = torch.tensor(self.decay, dtype=torch.float64).to(torch.float32).to(rt.device)
+        self.norm_w = rt.vector(tensors["norm"]) if self.has_norm_w else None
         self._freq = rope_inv_freqs(self.rope_dims, self.rope_base, self.rope_dims).to(rt.device) \
             if self.rope_dims else None
 
@@ -220,10 +235,13 @@ class RetentionMixer(Mixer):
         rt, ops, b = ctx.rt, ctx.rt.ops, ctx.batch
         H, d, dv = self.H, self.d, self.dv
         proj = ops.linear(h, self.w_in, None, torch.float32)               # [v | k | q | g]
-        ops.rotate_heads(proj, b.positions, self._freq, self.rope_dims, H, d, H * dv, d ** -0.5, H * dv + H * d, 1.0)
+        if self.turns:
+            ops.rotate_heads(proj, b.positions, self._freq, self.rope_dims, H, d, H * dv, self.key_scale, H * dv + H * d, 1.0)
+        extra = {"silu_inputs": True} if self.silu else {}
         o = ops.ssm_scan(proj[:, :H * dv + 2 * H * d], None, None, None, None, ctx.state(call, "retention"), b, H, dv,
-                         d, H, fixed_decay=self._decay)
-        g = ops.gated_rmsnorm(o, proj[:, H * dv + 2 * H * d:], None, H, self.eps, "silu_after", rt.dtype)
+                         d, H, fixed_decay=self._decay, **extra)
+        g = ops.gated_rmsnorm(o, proj[:, H * dv + 2 * H * d:], self.norm_w, 1 if self.norm_all else H, self.eps,
+                              f"{self.gate}_after", rt.dtype)
         ops.linear_add(g, self.w_o, resid)
 
 

@@ -73,6 +73,42 @@ class RotaryScaledNeoX(RotaryNeoX):
         return self._table, self.rotary_dim
 
 
+def yarn_blend(base: float, dims: int, factor: float, original: float, fast: float, slow: float) -> list[float]:
+    """Frequencies ``base^(-2i / dims)`` of which the slow ones are divided by ``factor``, each in double precision.
+    The pair whose wave turns t times within ``original`` positions is ``turn(t) = dims ln(original / (2 pi t)) /
+    (2 ln base)``; pairs up to ``max(floor turn(fast), 0)`` keep their frequency, from ``min(ceil turn(slow), dims - 1)``
+    on they are divided, and in between the two are mixed linearly in the pair's number."""
+    def turn(t):
+        return dims * math.log(original / (2.0 * math.pi * t)) / (2.0 * math.log(base))
+
+    first, last = max(math.floor(turn(fast)), 0), min(math.ceil(turn(slow)), dims - 1)
+    out = []
+    for i in range(dims // 2):
+        f = base ** (-2.0 * i / dims)
+        mix = min(max((i - first) / max(last - first, 0.001), 0.0), 1.0)
+        out.append(f / factor * mix + f * (1.0 - mix))
+    return out
+
+
+class RotaryYarnNeoX(RotaryNeoX):
+    """Split-half rotary embedding whose table is ``yarn_blend``'s and whose sines and cosines are multiplied by
+    ``0.1 ln(factor) + 1`` (``scaling``: a dict with ``factor``, ``original``, ``fast``, ``slow``; None: the plain table
+    and no factor)."""
+
+    def __init__(self, head_dim: int, theta: float, rotary_dim: int | None = None, scaling: dict | None = None):
+        super().__init__(head_dim, theta, rotary_dim)
+        self.scaling = {k: float(scaling[k]) for k in ("factor", "original", "fast", "slow")} if scaling else None
+        if self.scaling:
+            self.amplitude = 0.1 * math.log(self.scaling["factor"]) + 1.0
+
+    def rotary(self, rt: Runtime):
+        if self._table is None or self._table.device != rt.device:
+            f = yarn_blend(self.theta, self.rotary_dim, **self.scaling) if self.scaling else \
+                [self.theta ** (-2.0 * i / self.rotary_dim) for i in range(self.rotary_dim // 2)]
+            self._table = torch.tensor(f, dtype=torch.float64).to(torch.float32).to(rt.device)
+        return self._table, self.rotary_dim
+
+
 class RotaryInterleaved(RotaryNeoX):
     """The same rotation on neighbouring pairs ``(2i, 2i + 1)`` of every head."""
 
@@ -104,5 +140,6 @@ class LearnedPositions(PositionEncoding):
 register_part("position", "learned", LearnedPositions)
 register_part("position", "rope_neox", RotaryNeoX)
 register_part("position", "rope_scaled_neox", RotaryScaledNeoX)
+register_part("position", "rope_yarn_neox", RotaryYarnNeoX)
 register_part("position", "rope_interleaved", RotaryInterleaved)
 register_part("position", "none", NoPositionEncoding)

@@ -109,8 +109,11 @@ class PlainOps:
             v = v * (gate / (1.0 + torch.exp(-gate)))
         return v.to(out_dtype)
 
-    def ssm_scan(self, xbc, dt_raw, dt_bias, A_log, D, state, batch, heads, P, N, groups, fixed_decay=None):
+    def ssm_scan(self, xbc, dt_raw, dt_bias, A_log, D, state, batch, heads, P, N, groups, fixed_decay=None,
+                 silu_inputs=False):
         T = xbc.shape[0]
+        if silu_inputs:
+            xbc = xbc / (1.0 + torch.exp(-xbc))
         inner = heads * P
         y = torch.zeros((T, inner), dtype=torch.float32, device=xbc.device)
         cu, slots = batch.cu_q.tolist(), batch.state_slot.tolist()
@@ -291,8 +294,10 @@ class PlainOps:
         return out
 
     def head_norm_rope_write(self, qkv, positions, qn_w, kn_w, eps, inv_freq, rot_dims, interleaved, slots, k_cache,
-                             v_cache, nh, nkv, d, dv, D, out_dtype):
+                             v_cache, nh, nkv, d, dv, D, out_dtype, amplitude=1.0, norm_after=False):
         T = qkv.shape[0]
+        if slots is None:
+            nkv = 0
         Q, K = nh * d, nkv * d
         q, k = qkv[:, :Q].reshape(T, nh, d), qkv[:, Q:Q + K].reshape(T, nkv, d)
         v = qkv[:, Q + K:Q + K + nkv * dv].reshape(T, nkv, dv)
@@ -303,6 +308,12 @@ class PlainOps:
         if rot_dims:
             rotate = self._rotate_neighbours if interleaved else self._rotate
             q, k = rotate(q, positions, inv_freq, rot_dims), rotate(k, positions, inv_freq, rot_dims)
+            if amplitude != 1.0:
+                q[..., :rot_dims] *= amplitude
+                k[..., :rot_dims] *= amplitude
+        if norm_after:
+            q = q / torch.sqrt((q * q).mean(-1, keepdim=True) + eps)
+            k = k / torch.sqrt((k * k).mean(-1, keepdim=True) + eps)
         pad = torch.nn.functional.pad
         if slots is not None:
             ps = k_cache.shape[2]
@@ -375,6 +386,23 @@ class PlainOps:
 
     def linear_add(self, a, w, resid):
         resid += _f(a) @ _f(w).T
+
+    def layer_norm(self, x, w, b, eps, out_dtype, rows=None):
+        if rows is not None:
+            x = x[rows.long()]
+        c = x - x.mean(-1, keepdim=True)
+        return (c / torch.sqrt((c * c).mean(-1, keepdim=True) + eps) * w + b).to(out_dtype)
+
+    def post_norm_add(self, resid, y, w, b, eps, out_dtype, clear=False):
+        resid += self.layer_norm(y, w, b, eps, torch.float32) if b is not None else \
+            y / torch.sqrt((y * y).mean(-1, keepdim=True) + eps) * w
+        if clear:
+            y.zero_()
+        return resid if out_dtype == torch.float32 else resid.to(out_dtype)
+
+    def linear_glu(self, a, w_gate_up, act):
+        acc = _f(a) @ _f(w_gate_up).T
+        return (self.activation(acc[:, 0::2], act, torch.float32) * acc[:, 1::2]).to(a.dtype)
 
     @staticmethod
     def _swiglu(acc, dtype):
