@@ -13,6 +13,7 @@ continuous-batching workload on the windowed variant of the model (`serving`).
     python bench.py --workload zasazen      # the Zasazen design beside Qwen2-MoE at equal sizes, and its kernels alone
     python bench.py --workload salolorn     # the Salolorn design beside a dense Qwen2 at equal sizes, and its kernels alone
     python bench.py --workload faguzen      # the Faguzen design beside Qwen2-MoE at equal sizes, and its kernels alone
+    python bench.py --workload zepilorn     # the Zepilorn design beside a dense Qwen2 at equal sizes, and its kernels alone
 
 A step is one decode step of the whole batch.  One JSON line is printed.
 """
@@ -1310,6 +1311,209 @@ def run_faguzen(args, pk) -> dict:
     return out
 
 
+def zepilorn_config(width, vocab=32768, window=1024):
+    """Five layers of the design at a real model's layer sizes: attention heads of 128 (four query heads a key/value
+    head, half of each head rotated with a blended table) over a window, a 512-wide latent with 128-wide heads over
+    the same window, linear attention with heads of 64 x 128, attention on the first layer's keys and values, the
+    latent once more; a gated feed-forward three times the width."""
+    heads = width // 128
+    dense = {"kind": "dense", "ff": 3 * width}
+    att = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+           "mask": {"size": window}, "rot": {"base": 1e6, "dims": 64, "scaling": {"factor": 4.0, "original": 8192,
+                                                                                   "fast": 32.0, "slow": 1.0}}}
+    lat = {"heads": heads, "dim": 128, "vdim": 128, "kv_rank": 512, "scale": 128 ** -0.5, "mask": {"size": window}}
+    lin = {"heads": heads, "dim": 64, "vdim": 128, "decay": [1.0 - 2.0 ** (-5 - 5 * i / max(heads - 1, 1)) for i in range(heads)]}
+    layers = [{"type": t, "mixer": m, "mlp": dense} for t, m in
+              (("attention", att), ("latent_attention", lat), ("lightning", lin), ("attention", dict(att, kv_from=0)),
+               ("latent_attention", lat))]
+    return {"architecture": "Zepilorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "max_positions": 8192,
+            "layers": layers}
+
+
+def qwen_config_like_zepilorn(z):
+    """A dense Qwen2 (the Qwen2-MoE class with no experts) with the same width, vocabulary, layers, feed-forward, and
+    attention heads of the same number and size over the same window in every layer."""
+    att = z["layers"][0]["mixer"]
+    return dict(architectures=["Qwen2MoeForCausalLM"], model_type="qwen2_moe", num_hidden_layers=len(z["layers"]),
+                hidden_size=z["width"], num_attention_heads=att["heads"], num_key_value_heads=att["kv_heads"],
+                head_dim=att["dim"], num_experts=0, intermediate_size=z["layers"][0]["mlp"]["ff"], vocab_size=z["vocab"],
+                rope_theta=1e6, rms_norm_eps=1e-6, use_sliding_window=True, sliding_window=att["mask"]["size"],
+                max_window_layers=0, tie_word_embeddings=False, max_position_embeddings=8192)
+
+
+def zepilorn_kernels(z, pk, batch, context, prefill_tokens):
+    """Each kernel of the design alone at the layer sizes of `z`, beside the like kernel of an existing model at the
+    same sizes: a prompt of `prefill_tokens` tokens of one request, and a decode step of `batch` requests at `context`
+    tokens.  Microseconds (median of 5, the cache flushed before each), the bytes the kernel has to move at least,
+    and that over time over the measured copy bandwidth; attentions and products also with their flops."""
+    from types import SimpleNamespace
+
+    import torch
+
+    from dlm_b200.ops import native_ops
+    ops = native_ops(fast=True)
+    dev = "cuda"
+    W = z["width"]
+    att, ml, lin = (z["layers"][i]["mixer"] for i in (0, 1, 2))
+    ff = z["layers"][0]["mlp"]["ff"]
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    i32 = dict(dtype=torch.int32, device=dev)
+    bf = torch.bfloat16
+    rows = {}
+
+    def timed(name, case, fn, nbytes, flop=None):
+        ts = []
+        for _ in range(6):
+            _flush(torch, flush)
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record()
+            fn()
+            e1.record()
+            torch.cuda.synchronize()
+            ts.append(e0.elapsed_time(e1))
+        us = statistics.median(ts[1:]) * 1e3
+        row = {"us": round(us, 1), "mbytes": round(nbytes / 1e6, 2),
+               "frac_of_copy": round(nbytes / (us * 1e-6) / 1e9 / pk["hbm_gbs"], 3)}
+        if flop is not None:
+            row["gflop"] = round(flop / 1e9, 2)
+            row["frac_of_bf16_peak"] = round(flop / (us * 1e-6) / (pk["bf16_tflops"] * 1e12), 4)
+        rows.setdefault(name, {})[case] = row
+
+    for case, lens, start in (("prefill", [prefill_tokens], 0), ("decode", [1] * batch, context)):
+        T, R = sum(lens), len(lens)
+        cu = [0]
+        for n in lens:
+            cu.append(cu[-1] + n)
+        b = SimpleNamespace(num_requests=R, cu_q=torch.tensor(cu, **i32), state_slot=torch.arange(R, **i32),
+                            token_req=torch.tensor([r for r, n in enumerate(lens) for _ in range(n)], **i32),
+                            positions=torch.tensor([start + i for n in lens for i in range(n)], **i32))
+        held = start + max(lens)
+        b.max_kv_len = held
+        pages_each = -(-held // 64)
+        table = torch.arange(R * pages_each, **i32).reshape(R, pages_each)
+        slots = torch.cat([table[r, (start + torch.arange(n, device=dev)) // 64] * 64 + (start + torch.arange(n, device=dev)) % 64
+                           for r, n in enumerate(lens)]).to(torch.int32)
+        kv_len = torch.tensor([start + n for n in lens], **i32)
+        single = sum(1 for n in lens if n == 1)
+        # ---- norms behind a sublayer
+        resid, y = torch.randn(T, W, device=dev), torch.randn(T, W, device=dev)
+        wv, bv = torch.randn(W, device=dev) * 0.1, torch.randn(W, device=dev) * 0.1
+        timed("post_norm_add (closing norm, add, rounded copy, rows cleared)", case,
+              lambda: ops.post_norm_add(resid, y, wv, bv, 1e-6, bf, clear=True), T * W * 18)
+        timed("norm_add_norm (Salolorn's closing norm, add, opening norm)", case,
+              lambda: ops.norm_add_norm(resid, y, wv, wv, 1e-6, bf), T * W * 14)
+        timed("layer_norm", case, lambda: ops.layer_norm(resid, wv, bv, 1e-6, bf), T * W * 6)
+        timed("rmsnorm (Qwen2's)", case, lambda: ops.rmsnorm(resid, wv, 1e-6, bf), T * W * 6)
+        # ---- feed-forward with its gate in the product's epilogue
+        h = torch.randn(T, W, device=dev).to(bf)
+        wgu = (torch.randn(2 * ff, W, device=dev) * 0.02).to(bf)
+        for name, act in (("gate and up product, gelu (tanh form)", "gelu_tanh"), ("gate and up product, silu (Qwen2's)", "silu")):
+            timed(name, case, lambda: ops.linear_glu(h, wgu, act), (2 * ff * W + T * (W + ff)) * 2, flop=4.0 * T * W * ff)
+        # ---- attention over a window with a silent sink
+        Ha, Ga, d, dv = att["heads"], att["kv_heads"], att["dim"], att["vdim"]
+        D = max(d, dv)
+        window = att["mask"]["size"]
+        rd = att["rot"]["dims"]
+        k_cache = (torch.randn(R * pages_each + 1, Ga, 64, D, device=dev) * 0.3).to(bf)
+        v_cache = (torch.randn(R * pages_each + 1, Ga, 64, D, device=dev) * 0.3).to(bf)
+        aq = torch.randn(T, (Ha + Ga) * d + Ga * dv, device=dev)
+        freq = torch.tensor([att["rot"]["base"] ** (-2.0 * i / rd) for i in range(rd // 2)], device=dev)
+        nw = torch.randn(d, device=dev)
+        io = T * ((Ha + Ga) * d + Ga * dv) * 4 + T * (Ha + 2 * Ga) * D * 2
+        timed("head_norm_rope_write, norm behind the rotation", case,
+              lambda: ops.head_norm_rope_write(aq, b.positions, None, None, 1e-6, freq, rd, False, slots, k_cache, v_cache,
+                                               Ha, Ga, d, dv, D, bf, amplitude=1.14, norm_after=True), io)
+        timed("head_norm_rope_write, norm behind the rotation, queries only", case,
+              lambda: ops.head_norm_rope_write(aq, b.positions, None, None, 1e-6, freq, rd, False, None, k_cache, v_cache,
+                                               Ha, Ga, d, dv, D, bf, amplitude=1.14, norm_after=True), T * Ha * (d * 4 + D * 2))
+        timed("head_norm_rope_write, norm before it (Salolorn's)", case,
+              lambda: ops.head_norm_rope_write(aq, b.positions, nw, nw, 1e-6, freq, rd, False, slots, k_cache, v_cache,
+                                               Ha, Ga, d, dv, D, bf), io)
+        ffreq = torch.tensor([1e6 ** (-2.0 * i / D) for i in range(D // 2)], device=dev)
+        timed("rope_kv_write (Qwen2's)", case,
+              lambda: ops.rope_kv_write(aq, b.positions, ffreq, D, slots, k_cache, v_cache, Ha, Ga, D, bf), io)
+        q = ops.head_norm_rope_write(aq, b.positions, None, None, 1e-6, freq, rd, False, slots, k_cache, v_cache, Ha, Ga, d,
+                                     dv, D, bf, norm_after=True)
+        keys = sum(min(window, start + i + 1) for n in lens for i in range(n))
+        span = min(window, held)
+        nbytes = (R * span if case == "decode" else held) * Ga * D * 4 + T * Ha * D * 4
+        zero = torch.zeros(Ha, device=dev)
+        for name, sk in (("attention over a window with a sink", zero), ("attention over a window (Qwen2's)", None)):
+            timed(name, case, lambda: ops.attention(q, k_cache, v_cache, table, b.cu_q, kv_len, window, att["scale"], Ha, Ga, D,
+                                                    max(lens), held, single, sinks=sk), nbytes, flop=4.0 * keys * Ha * D)
+        # ---- latent attention without positions
+        Hl, dn, dvl, rank, lw = ml["heads"], ml["dim"], ml["vdim"], ml["kv_rank"], ml["mask"]["size"]
+        keys = sum(min(lw, start + i + 1) for n in lens for i in range(n))
+        for dr, who in ((0, ""), (64, " (Zesapel's: 64 rotated entries more, a sink)")):
+            cache = (torch.randn(R * pages_each + 1, 1, 64, rank + dr, device=dev) * 0.3).to(bf)
+            qc = Hl * (dn + dr)
+            lp = torch.randn(T, qc + rank + dr, device=dev)
+            kvn = torch.randn(rank, device=dev)
+            lf = torch.ones(max(dr // 2, 1), device=dev)
+            sk = torch.zeros(Hl, device=dev) if dr else None
+            timed("latent_prep" + who, case,
+                  lambda: ops.latent_prep(lp, 0, 0, None, qc, rank, kvn, dr, lf, dr, b.positions, slots, 1e-6, cache, bf),
+                  T * (rank + dr) * 6)
+            timed("latent_q_split" + who, case,
+                  lambda: ops.latent_q_split(lp[:, :qc], b.positions, lf, dr, Hl, dn, dr, bf), T * Hl * ((dn + dr) * 4 + dn * 2 + dr * 4))
+            qpl, q_rot = ops.latent_q_split(lp[:, :qc], b.positions, lf, dr, Hl, dn, dr, bf)
+            wukT = (torch.randn(Hl, rank, dn, device=dev) * 0.05).to(bf)
+            wuv = (torch.randn(Hl, dvl, rank, device=dev) * 0.05).to(bf)
+            offs = ops.head_offsets(Hl, T, dev)
+            q_lat = ops.grouped_linear(qpl.reshape(Hl * T, dn), wukT, offs).reshape(Hl, T, rank)
+            timed("latent_attention" + who, case,
+                  lambda: ops.latent_attention(q_lat, q_rot, sk, cache, table, b, Hl, dr, rank, lw, ml["scale"]),
+                  (R * min(lw, held) if case == "decode" else held) * (rank + dr) * 2 + T * Hl * (rank * 6 + dr * 4),
+                  flop=2.0 * keys * Hl * (2 * rank + dr))
+            if dr == 0:
+                lat = ops.latent_attention(q_lat, q_rot, sk, cache, table, b, Hl, dr, rank, lw, ml["scale"])
+                timed("queries through W_uk (grouped product)", case,
+                      lambda: ops.grouped_linear(qpl.reshape(Hl * T, dn), wukT, offs),
+                      Hl * (T * dn * 2 + rank * dn * 2 + T * rank * 4))
+                timed("latents through W_uv (grouped product)", case,
+                      lambda: ops.grouped_linear(lat.reshape(Hl * T, rank), wuv, offs),
+                      Hl * (T * rank * 2 + rank * dvl * 2 + T * dvl * 4))
+                val = ops.grouped_linear(lat.reshape(Hl * T, rank), wuv, offs)
+                timed("latent_gate_out (no gate)", case, lambda: ops.latent_gate_out(val, None, Hl, dvl, bf), T * Hl * dvl * 6)
+        # ---- linear attention with constant decays on activated inputs
+        H2, d2, dv2 = lin["heads"], lin["dim"], lin["vdim"]
+        rp = torch.randn(T, H2 * dv2 + 2 * H2 * d2, device=dev)
+        decay = torch.tensor(lin["decay"], device=dev)
+        rst = torch.zeros(R + 1, H2, d2, dv2, device=dev)
+        sb = T * (H2 * dv2 * 2 + 2 * H2 * d2) * 4 + 2 * R * H2 * d2 * dv2 * 4
+        for name, silu in (("ssm_scan with constant decays, silu on its inputs", True),
+                           ("ssm_scan with constant decays (Zasazen's retention)", False)):
+            timed(name, case, lambda: ops.ssm_scan(rp, None, None, None, None, rst, b, H2, dv2, d2, H2, fixed_decay=decay,
+                                                   silu_inputs=silu), sb)
+        o_, g_, n2 = torch.randn(T, H2 * dv2, device=dev), torch.randn(T, H2 * dv2, device=dev), torch.randn(H2 * dv2, device=dev)
+        timed("gated_rmsnorm, all heads together, sigmoid gate", case,
+              lambda: ops.gated_rmsnorm(o_, g_, n2, 1, 1e-6, "sigmoid_after", bf), T * H2 * dv2 * 10)
+        timed("gated_rmsnorm, per head, silu gate (Salolorn's)", case,
+              lambda: ops.gated_rmsnorm(o_, g_, n2, H2, 1e-6, "silu_after", bf), T * H2 * dv2 * 10)
+    ops.check_errors()
+    return rows
+
+
+def run_zepilorn(args, pk) -> dict:
+    sampler = ClockSampler()
+    sampler.start()
+    t0 = time.time()
+    out = {"workload": "zepilorn", "dtype": "bf16", "data": "synthetic: seeded uniform token ids, random weights N(0, 0.02)",
+           "peaks": pk, "sizes": {}, "l2": "a buffer larger than L2 is written before every timed step"}
+    for width in (1024, 2048, 4096):
+        z = zepilorn_config(width)
+        q = qwen_config_like_zepilorn(z)
+        out["sizes"][str(width)] = {
+            "layers": len(z["layers"]), "zepilorn": measure_engine(z, args.batch, args.prompt_len, args.steps, 2048),
+            "qwen2_dense": measure_engine(q, args.batch, args.prompt_len, args.steps, 2048)}
+    out["kernels_width_2048"] = zepilorn_kernels(zepilorn_config(2048), pk, args.batch, args.prompt_len, 2048)
+    t1 = time.time()
+    time.sleep(0.2)
+    sampler.stop()
+    out["clocks"] = sampler.summary(t0, t1)
+    return out
+
+
 def layers_that_fit(raw, want, reserve_gb=40.0):
     """As many layers of `raw` (at most `want`) as the free device memory holds beside `reserve_gb` for
     the cache pool, the head, graphs and activations."""
@@ -1369,7 +1573,8 @@ def main() -> int:
     ap.add_argument("--no-points", action="store_true", help="skip the batch 1 / 64 and prefill measurements")
     ap.add_argument("--no-extras", action="store_true", help="skip `sizes_57b` and `serving`")
     ap.add_argument("--only-prefill", action="store_true", help="measure the 2,048-token prefill alone (for profiles)")
-    ap.add_argument("--workload", default="decode", choices=["decode", "serving", "sweep", "kernels", "zesapel", "zasazen", "salolorn", "faguzen"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "serving", "sweep", "kernels", "zesapel", "zasazen", "salolorn", "faguzen",
+                                                              "zepilorn"],
                     help="serving: the continuous-batching workload on the windowed model, instead of the default line; "
                          "sweep: decode at contexts of 1k to 32k and prefill of longer prompts, a line of its own; "
                          "kernels: the weight-streaming product alone")
@@ -1411,6 +1616,9 @@ def main() -> int:
         return 0
     if args.workload == "faguzen":
         print(json.dumps(run_faguzen(args, pk)))
+        return 0
+    if args.workload == "zepilorn":
+        print(json.dumps(run_zepilorn(args, pk)))
         return 0
     max_batch = 64 if not args.no_points else args.batch
     m = Measurement(MODEL, args.layers, args.prompt_len, args.context, max_batch, pk, page=args.page_size)

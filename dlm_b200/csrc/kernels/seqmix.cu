@@ -298,6 +298,69 @@ __global__ void gated_rmsnorm_kernel(const float* __restrict__ y, int ldy, const
     }
 }
 
+// The same, modes 1 and 2, for wide groups (a multiple of four entries): a thread keeps V groups of four neighbouring
+// entries of y and of the gate in registers, all loads in flight before the sum.
+template <typename TOut, int V>
+__global__ void gated_rmsnorm_wide_kernel(const float* y, int ldy, const float* gate, int ldg,
+                                          const float* __restrict__ w, TOut* out, int ldo, int gs, float eps, int mode) {
+    dep_wait();          // nothing is read or written before the kernels before this one have ended
+    dep_launch_next();
+    __shared__ float s_part[32];
+    const int t = blockIdx.x, g = blockIdx.y;
+    const float* yr = y + (long long)t * ldy + (long long)g * gs;
+    const float* gr = gate + (long long)t * ldg + (long long)g * gs;
+    float4 a[V], b[V];
+    float part = 0.f;
+#pragma unroll
+    for (int u = 0; u < V; ++u) {
+        const int i = 4 * (threadIdx.x + u * blockDim.x);
+        a[u] = b[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (i < gs) {
+            a[u] = *reinterpret_cast<const float4*>(yr + i);
+            b[u] = *reinterpret_cast<const float4*>(gr + i);
+        }
+    }
+#pragma unroll
+    for (int u = 0; u < V; ++u) {
+        part = fmaf(a[u].x, a[u].x, part);
+        part = fmaf(a[u].y, a[u].y, part);
+        part = fmaf(a[u].z, a[u].z, part);
+        part = fmaf(a[u].w, a[u].w, part);
+    }
+    const float inv = 1.0f / sqrtf(block_sum(part, s_part) / (float)gs + eps);
+    auto gated = [&](float v, float z, float wi) { return ((v * inv) * wi) * (mode == 1 ? sigmoid_f(z) : silu_f(z)); };
+#pragma unroll
+    for (int u = 0; u < V; ++u) {
+        const int i = 4 * (threadIdx.x + u * blockDim.x);
+        if (i >= gs) continue;
+        const float4 ww = w != nullptr ? *reinterpret_cast<const float4*>(w + (long long)g * gs + i)
+                                       : make_float4(1.f, 1.f, 1.f, 1.f);
+        TOut* o = out + (long long)t * ldo + (long long)g * gs + i;
+        o[0] = from_f32<TOut>(gated(a[u].x, b[u].x, ww.x));
+        o[1] = from_f32<TOut>(gated(a[u].y, b[u].y, ww.y));
+        o[2] = from_f32<TOut>(gated(a[u].z, b[u].z, ww.z));
+        o[3] = from_f32<TOut>(gated(a[u].w, b[u].w, ww.w));
+    }
+}
+
+template <typename TOut>
+bool launch_gated_rmsnorm_wide(const float* y, int ldy, const float* gate, int ldg, const float* w, void* out, int ldo,
+                               int T, int groups, int gs, float eps, int mode, cudaStream_t stream) {
+    const uintptr_t all = reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(w);
+    if (mode == 0 || gs < 512 || gs > 8192 || gs % 4 != 0 || ldy % 4 != 0 || ldg % 4 != 0 || all % 16 != 0) return false;
+    const int quads = gs / 4, threads = quads >= 256 ? 256 : (quads + 31) / 32 * 32;
+    const int v = (quads + threads - 1) / threads;
+#define DLM_GW(V)                                                                                                      \
+    launch_dep(gated_rmsnorm_wide_kernel<TOut, V>, dim3(T, groups), dim3(threads), 0, stream, y, ldy, gate, ldg, w,     \
+               static_cast<TOut*>(out), ldo, gs, eps, mode)
+    if (v <= 1) DLM_GW(1);
+    else if (v <= 2) DLM_GW(2);
+    else if (v <= 4) DLM_GW(4);
+    else DLM_GW(8);
+#undef DLM_GW
+    return true;
+}
+
 // ------------------------------------------------------------ pieces of the two scans
 // Four bytes from global to shared memory without a register in between; a group of such copies is waited for
 // with copies_wait<N>() (all but the N newest groups have landed).
@@ -753,6 +816,13 @@ void gated_rmsnorm(const float* y, int ldy, const float* gate, int ldg, const fl
                    cudaStream_t stream) {
     if (T <= 0) return;
     DLM_CHECK(row_scale == nullptr || mode != 0, "gated_rmsnorm: a factor per row goes with a gate after the norm");
+    if (row_scale == nullptr &&
+        (out_dtype == F32 ? launch_gated_rmsnorm_wide<float>(y, ldy, gate, ldg, w, out, ldo, T, groups, group_size, eps, mode, stream)
+                          : launch_gated_rmsnorm_wide<__nv_bfloat16>(y, ldy, gate, ldg, w, out, ldo, T, groups, group_size,
+                                                                     eps, mode, stream))) {
+        check_launch("gated_rmsnorm (wide groups)");
+        return;
+    }
     const int threads = group_size >= 256 ? 256 : (group_size >= 128 ? 128 : (group_size > 32 ? 64 : 32));
     if (out_dtype == F32)
         launch_dep(gated_rmsnorm_kernel<float>, dim3(T, groups), dim3(threads), 0, stream, y, ldy, gate, ldg, w, static_cast<float*>(out),
