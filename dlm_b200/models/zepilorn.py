@@ -1,7 +1,7 @@
 """Zepilorn as a ``ModelSpec`` of parts.
 
 Token embedding and a separate head; a centred norm with weight and bias on the *output* of every sublayer (and before
-the head), followed by a learned scale per entry; the sublayers read the residual itself.  Mixers: grouped-query
+the head), followed by a learned scale per entry; a sublayer's input is not normed.  Mixers: grouped-query
 attention over a window (a rotation over part of each head whose slow waves are slowed further and whose sines and
 cosines are scaled; queries and keys divided by their root mean square after it; a softmax with one more in its
 denominator) that may read the keys and values of an earlier layer; attention over a window through one normed latent

@@ -142,8 +142,8 @@ class SandwichBlock(ParallelBlock):
 
 
 class PostNormBlock(ParallelBlock):
-    """Norms on the sublayers' outputs only: ``x += s1 * norm1(mixer(x))``, then ``x += s2 * norm2(ffn(x))``; the sublayers
-    read x itself.  ``layer_scale``: the learned scales ``s1`` and ``s2`` (``[hidden_size]``) exist; they join the norms'
+    """What a sublayer puts out is normed, what it takes in is not: ``x += s1 * norm1(mixer(x))``, then
+    ``x += s2 * norm2(ffn(x))``.  ``layer_scale``: the learned scales ``s1`` and ``s2`` (``[hidden_size]``) exist; they join the norms'
     weights at load.  ``ffn`` None: only the first sublayer.
 
     A sublayer adds its output into rows of zeros.  Where the norm lets a kernel apply it (``Norm.closing``), the norm,

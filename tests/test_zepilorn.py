@@ -418,3 +418,19 @@ def test_norm_on_outputs_with_other_norms_and_blocks():
         assert float(ctx.take_zeroed(x).abs().max()) == 0.0
     with pytest.raises(NotImplementedError):
         build_part("norm", PartSpec("dynamic_tanh", {"size": W})).scale_output(torch.ones(W))
+
+
+def test_the_benchmarks_configurations_resolve():
+    """The benchmark's model of this design and the one beside it: equal width, layers, feed-forward and attention
+    heads; the reader's layer owns no cache."""
+    import sys as _sys
+    _sys.path.insert(0, os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
+    import bench
+    from dlm_b200.registry import resolve
+    z = bench.zepilorn_config(1024)
+    _, cfg, spec = resolve(copy.deepcopy(z))
+    _, q, qspec = resolve(bench.qwen_config_like_zepilorn(z))
+    assert len(spec.layers) == len(qspec.layers) == 5 and spec.hidden_size == qspec.hidden_size == 1024
+    att = cfg.layers[0]["mixer"]
+    assert (q.num_attention_heads, q.num_key_value_heads, q.head_dim) == (att["heads"], att["kv_heads"], att["dim"])
+    assert spec.order[3].reads_cache_of == 0
