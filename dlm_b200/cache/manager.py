@@ -8,8 +8,8 @@ A mixer declares what it caches per token as a list of tensors (keys and values
 for attention; a mixer with one latent vector per token declares one).  Layout
 of each: ``[pages + 1, heads, page_size, width]``; a page of one head is a
 contiguous ``page_size x width`` tile.  The last page is a sink that padded rows
-write to; the pool never hands it out.  Calls whose window and page size agree
-form a group with one pool of page ids and one block table per request.
+write to; the pool never hands it out.  Calls whose window, kept first tokens
+and page size agree form a group with one pool of page ids and one block table per request.
 """
 from __future__ import annotations
 
@@ -35,7 +35,7 @@ class ModelCache:
         self.num_pages = int(num_pages)
         self.num_slots = int(num_slots)
         needs = model.cache_needs()
-        # groups: one per distinct (window, page size) among the calls that own paged tensors
+        # groups: one per distinct (window, page size, kept first tokens) among the calls that own paged tensors
         self.group_windows: list[int] = []
         self.group_page_size: list[int] = []
         self.group_pages: list[int] = []
@@ -44,16 +44,18 @@ class ModelCache:
         self.tensors: dict[int, dict[str, torch.Tensor]] = {}
         self.state: dict[int, torch.Tensor] = {}
         self.named_state: dict[tuple[int, str], torch.Tensor] = {}    # states of parts that declared several
-        keys: list[tuple[int, int]] = []
+        self.group_keep: list[int] = []          # first tokens a window's group keeps beside the window
+        keys: list[tuple[int, int, int]] = []
         for ci, (need, st, owner) in enumerate(needs):
             self.call_owner[ci] = owner
             if need is not None and owner == ci:
                 ps = int(need.page_size or self.page_size)
-                key = (int(need.window or 0), ps)
+                key = (int(need.window or 0), ps, int(need.keep_first) if need.window else 0)
                 if key not in keys:
                     keys.append(key)
                     self.group_windows.append(key[0])
                     self.group_page_size.append(ps)
+                    self.group_keep.append(key[2])
                     # the same number of tokens in every pool
                     self.group_pages.append(max(1, -(-self.num_pages * self.page_size // ps)))
                 g = keys.index(key)
@@ -77,9 +79,11 @@ class ModelCache:
         if not self.group_windows:
             self.group_windows.append(0)     # a model without paged caches still counts tokens
             self.group_page_size.append(self.page_size)
+            self.group_keep.append(0)
             self.group_pages.append(self.num_pages)
         self.manager = host.CacheManager(
-            [host.GroupSpec(ps, w, n) for ps, w, n in zip(self.group_page_size, self.group_windows, self.group_pages)],
+            [host.GroupSpec(ps, w, n, k) for ps, w, n, k in zip(self.group_page_size, self.group_windows,
+                                                                self.group_pages, self.group_keep)],
             self.num_slots)
         self._pinned = []
         self._ring = 0

@@ -15,12 +15,14 @@ PYBIND11_MODULE(_dlm_host, m) {
     py::register_exception<CacheExhausted>(m, "CacheExhausted", PyExc_RuntimeError);
 
     py::class_<GroupSpec>(m, "GroupSpec")
-        .def(py::init([](int page_size, int window, int num_pages) {
-                 GroupSpec g; g.page_size = page_size; g.window = window; g.num_pages = num_pages; return g;
-             }), py::arg("page_size"), py::arg("window"), py::arg("num_pages"))
+        .def(py::init([](int page_size, int window, int num_pages, int keep_first) {
+                 GroupSpec g; g.page_size = page_size; g.window = window; g.num_pages = num_pages; g.keep_first = keep_first;
+                 return g;
+             }), py::arg("page_size"), py::arg("window"), py::arg("num_pages"), py::arg("keep_first") = 0)
         .def_readwrite("page_size", &GroupSpec::page_size)
         .def_readwrite("window", &GroupSpec::window)
-        .def_readwrite("num_pages", &GroupSpec::num_pages);
+        .def_readwrite("num_pages", &GroupSpec::num_pages)
+        .def_readwrite("keep_first", &GroupSpec::keep_first);
 
     py::class_<GroupStats>(m, "GroupStats")
         .def_readonly("total_pages", &GroupStats::total_pages)

@@ -16,6 +16,7 @@ CacheManager::CacheManager(std::vector<GroupSpec> groups, int num_slots) : group
         const GroupSpec& s = groups_[g];
         if (s.page_size <= 0) throw std::invalid_argument("page_size must be > 0");
         if (s.window < 0) throw std::invalid_argument("window must be >= 0");
+        if (s.keep_first < 0) throw std::invalid_argument("keep_first must be >= 0");
         if (s.num_pages < 0) throw std::invalid_argument("num_pages must be >= 0");
         std::vector<int32_t> fl(s.num_pages);
         // low ids are handed out first: the stack's top is page 0
@@ -69,6 +70,8 @@ int CacheManager::first_needed_page(int g, int next_pos) const {
     return lo / s.page_size;
 }
 
+int CacheManager::kept_pages(int g) const { return ceil_div(groups_[g].keep_first, groups_[g].page_size); }
+
 std::vector<int> CacheManager::pages_needed(int slot, int n) const {
     if (!is_open(slot)) throw std::invalid_argument("pages_needed: slot is not open");
     if (n < 0) throw std::invalid_argument("pages_needed: n must be >= 0");
@@ -82,7 +85,7 @@ std::vector<int> CacheManager::pages_needed(int slot, int n) const {
         int give = 0;
         if (n > 0) {
             const int upto = std::min(first_needed_page((int)g, sl.length), have);
-            for (int i = sl.first_live[g]; i < upto; ++i)
+            for (int i = std::max(sl.first_live[g], kept_pages((int)g)); i < upto; ++i)
                 if (sl.tables[g][i] >= 0) ++give;
         }
         need[g] = take - give;
@@ -134,7 +137,7 @@ void CacheManager::append(const std::vector<std::pair<int, int>>& slot_and_n) {
         Slot& sl = slots_[sn.first];
         for (size_t g = 0; g < groups_.size(); ++g) {
             const int upto = std::min(first_needed_page((int)g, sl.length), (int)sl.tables[g].size());
-            for (int i = sl.first_live[g]; i < upto; ++i) {
+            for (int i = std::max(sl.first_live[g], kept_pages((int)g)); i < upto; ++i) {
                 if (sl.tables[g][i] >= 0) {
                     free_[g].push_back(sl.tables[g][i]);
                     sl.tables[g][i] = -1;

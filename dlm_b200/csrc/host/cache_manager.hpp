@@ -4,8 +4,9 @@
 // Python side keeps the tensors those ids index.  Layers with the same cache
 // needs form a *group*; each group has a pool of pages of its own and each
 // request has one block table per group.  A group either keeps every key
-// (window == 0) or only the last `window` positions; in the second case a page
-// goes back to the pool as soon as no later query can see any of its positions.
+// (window == 0) or only the last `window` positions and the first `keep_first`;
+// in the second case a page goes back to the pool as soon as no later query can
+// see any of its positions.
 //
 // Behaviour mirrored from the reference's bookkeeping (src/cache/paged.rs):
 // a LIFO free list that hands out low ids first (:117-126); growth that is
@@ -24,6 +25,7 @@ struct GroupSpec {
     int page_size = 16;   // tokens per page
     int window = 0;       // 0: keep all keys; W > 0: a query at p sees keys j with p - j < W
     int num_pages = 0;    // pages in this group's pool
+    int keep_first = 0;   // with a window: a query also sees the positions below this
 };
 
 struct GroupStats {
@@ -119,6 +121,8 @@ private:
     };
     // first logical page that a query at position >= next_pos can still see
     int first_needed_page(int g, int next_pos) const;
+    // how many logical pages at the start hold a position that is kept whatever the window
+    int kept_pages(int g) const;
 
     std::vector<GroupSpec> groups_;
     std::vector<std::vector<int32_t>> free_;   // per group LIFO

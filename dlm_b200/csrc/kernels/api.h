@@ -15,7 +15,9 @@ enum Epilogue : int {
     EPI_SWIGLU = 2,   // out[m, n/2] = silu(acc[m, n]) * acc[m, n+1] for even n (interleaved weight rows)
     EPI_GELU = 3,     // out[m, n] = gelu(acc (+ bias[n])) in its exact (erf) form, stored as the output dtype
     EPI_GELU_TANH = 4,// the same with gelu in its tanh form: z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))) / 2
-    EPI_GEGLU_TANH = 5// EPI_SWIGLU with that gelu in place of silu
+    EPI_GEGLU_TANH = 5, // EPI_SWIGLU with that gelu in place of silu
+    EPI_CLAMP_GLU = 6 // out[m, n/2] = g sigmoid(alpha g) (u + shift), g = min(acc[m, n], limit), u = acc[m, n+1] clamped to
+                      // [-limit, limit]; `bias` points at the three constants {limit, alpha, shift} (f32)
 };
 
 // out[T, H] (f32) = table[tokens[t], :] * scale
@@ -61,12 +63,15 @@ void rope_kv_write(const float* qkv, const int32_t* positions, const float* inv_
 // floor(p / chunk) * chunk on (chunks are counted from a request's position 0).  sinks (f32 [nh]) != nullptr: the
 // softmax's denominator also holds exp(sinks[head]), unscaled, without key or value.  softcap c > 0: the scaled dot
 // product becomes c * tanh(dot * scale / c) before the distance term and the mask.
+// keep > 0 with a window: the first `keep` positions of a request stay visible (at their true positions).  parts 2:
+// query head h is zero outside half h % 2 of its hd entries, and kernels may leave that half of the product out.
 // num_single: how many requests have exactly one query token.  With fast != 0 and a scratch buffer of
 // attention_scratch_floats(...) floats those go to the split-key decode kernel.
 void attention(const void* q, const void* k_cache, const void* v_cache, const int32_t* block_table, int table_width,
                const int32_t* cu_q, const int32_t* kv_len, void* out, int T, int R, int nh, int nkv, int hd,
                int page_size, int total_pages, int window, float scale, const float* slopes, int chunk,
-               const float* sinks, float softcap, int max_q_len, int max_kv_len, int num_single, float* scratch, int dtype,
+               const float* sinks, float softcap, int keep, int parts, int max_q_len, int max_kv_len, int num_single,
+               float* scratch, int dtype,
                int fast, cudaStream_t stream);
 // Floats of scratch the decode kernel needs for a step of R requests whose longest holds max_kv_len tokens.
 size_t attention_scratch_floats(int R, int nh, int nkv, int hd, int max_kv_len);
@@ -101,7 +106,7 @@ int router_topk_permute(const void* h, const void* w, const float* norm_w, float
 void moe_permute(const int32_t* ids, int n, int k, int E, int32_t* offsets, int32_t* rows, int32_t* dest,
                  cudaStream_t stream);
 
-// resid[t, :] += sum_j wts[t, j] * y[dest[t, j], :] (+ shared_scale * gate[t] * shared[t, :]); gate == nullptr: 1.
+// resid[t, :] += sum_j wts[t, j] * y[dest[t, j], :] (+ shared_scale * gate[t] * shared[t, :]); wts, gate == nullptr: 1.
 // ids (i32 [T, k]) != nullptr: a pair whose expert id is num_real or more reads passthrough[t, :] (f32 [T, H]) in
 // place of its row of y (an expert that hands its input through; y may then be nullptr when num_real is 0).
 void moe_combine(const float* y, const int32_t* dest, const float* wts, const float* shared, const float* gate,
@@ -162,6 +167,10 @@ void streams_update_reduce(float* xs, const float* mix, const float* outw, const
 void causal_conv(const float* x, int ldx, const float* w, const float* bias, float* state, const int32_t* cu_q,
                  const int32_t* token_req, const int32_t* state_slot, int T, int R, int C, int taps, int add_input,
                  int act, void* out, int ldo, int out_dtype, cudaStream_t stream);
+// The second half of causal_conv alone: state <- the last taps - 1 of (carried inputs, this step's inputs) per request;
+// skip_single != 0: requests with one token are left as they are (whoever convolved has seen to them).
+void conv_state(const float* x, int ldx, float* state, const int32_t* cu_q, const int32_t* state_slot, int R, int C,
+                int taps, int skip_single, cudaStream_t stream);
 
 // out[r, c] = f(x[r, c]); op 0 tanh, 1 gelu (erf), 2 silu, 3 gelu (tanh form), 4 copy.  x f32, out in out_dtype.
 void activation(const float* x, int ldx, void* out, int ldo, int rows, int cols, int op, int out_dtype,
@@ -347,5 +356,25 @@ void layer_norm(const float* x, const int32_t* rows, const float* w, const float
 // (nullptr).  clear != 0: y is left all zeros (for the next sublayer, which adds into it).
 void post_norm_add(float* resid, float* y, const float* w, const float* b, float eps, int centered, int clear, void* out,
                    int T, int H, int out_dtype, cudaStream_t stream);
+
+// ---- heads that are the difference of two score maps, experts whose weight meets their input (diffmix.cu) ----
+
+// proj rows (f32) hold [q: H x 2 x d | k: G x 2 x d | v: G x dv | ...], map 1 then map 2 per head.  conv [taps, C] (f32,
+// C the channels of q, k and v; nullptr: none): every channel becomes sum_j conv[j] * its value taps - 1 - j tokens ago,
+// with state [slots, taps - 1, C] (f32) the inputs before a request's next token (zeros at its start), brought up to
+// date.  Then every map of q and k is divided by its root mean square over d and multiplied by qn / kn [d].  A stored
+// head is D wide: the two maps' keys fill its halves; q_out [T, 2H, D] holds map m's query in half m, zeros elsewhere;
+// k and v go to the token's slot of the paged caches [pages, G, page_size, D].
+void map_norm_write(const float* proj, int ld, const float* conv, int taps, float* state, const int32_t* cu_q,
+                    const int32_t* token_req, const int32_t* state_slot, const float* qn, const float* kn, float eps,
+                    const int32_t* slots, void* q_out, void* k_cache, void* v_cache, int T, int R, int num_single, int H,
+                    int G, int d, int dv, int D, int page_size, int total_pages, int dtype, cudaStream_t stream);
+// o [T, 2H, D] (two maps a head, dv entries each): out[t, h] = c / sqrt(mean(c^2) + eps) * factor * sigmoid(gate) with
+// c = o[t, 2h] - lambda * o[t, 2h + 1]; gate f32 [T, H * dv] raw (nullptr: none); out [T, H * dv] in `dtype`
+void diff_norm_gate(const void* o, const float* gate, int ldg, void* out, int T, int H, int dv, int D, float lambda,
+                    float eps, float factor, int dtype, cudaStream_t stream);
+// out[dest[t, j], :] = wts[t, j] * h[t, :]: the experts' rows side by side, each already weighted (h, out in `dtype`)
+void weigh_rows(const void* h, const float* wts, const int32_t* dest, void* out, int T, int k, int H, int dtype,
+                cudaStream_t stream);
 
 }  // namespace dlmk

@@ -15,9 +15,12 @@ size_t attention_scratch_floats(int R, int nh, int nkv, int hd, int max_kv_len) 
 void attention(const void* q, const void* k_cache, const void* v_cache, const int32_t* block_table, int table_width,
                const int32_t* cu_q, const int32_t* kv_len, void* out, int T, int R, int nh, int nkv, int hd,
                int page_size, int total_pages, int window, float scale, const float* slopes, int chunk,
-               const float* sinks, float softcap, int max_q_len, int max_kv_len, int num_single, float* scratch, int dtype,
+               const float* sinks, float softcap, int keep, int parts, int max_q_len, int max_kv_len, int num_single, float* scratch, int dtype,
                int fast, cudaStream_t stream) {
-    const Score score(scale, slopes, chunk, sinks, softcap);
+    // without a window every position is visible anyway
+    const Score score(scale, slopes, chunk, sinks, softcap, window > 0 ? keep : 0, parts);
+    DLM_CHECK(keep >= 0 && (keep == 0 || chunk <= 0), "attention: kept first positions go with a window, not with chunks");
+    DLM_CHECK(parts == 1 || (parts == 2 && nh % 2 == 0 && hd % 2 == 0), "attention: a stored head has one part or two halves");
     DLM_CHECK(softcap >= 0.f, "attention: a score cap is positive (0: none)");
     if (T <= 0 || R <= 0) return;
     DLM_CHECK(chunk >= 0, "attention: a chunk size is positive (0: none)");

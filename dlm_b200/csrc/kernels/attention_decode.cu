@@ -73,9 +73,10 @@ attention_decode_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
     if (scale.chunk > 0) lo = max(lo, (p / scale.chunk) * scale.chunk);       // a chunked mask: from the chunk's start
     // the request's own visible keys [lo, len) are cut into n_splits shares (multiples of 64 keys, at most
     // `chunk`), so that a request far shorter than the longest, or one with a window, still uses every block
-    int share = (len - lo + n_splits - 1) / n_splits;
+    const DecodeKeys keys(lo, len, scale.keep);                    // (below, j counts keys closed up; keys.at(j) is a position)
+    int share = (keys.end - keys.first + n_splits - 1) / n_splits;
     share = min(chunk, (share + 63) / 64 * 64);
-    const int j_begin = min(len, lo + sp * share), j_end = min(len, lo + (sp + 1) * share);
+    const int j_begin = min(keys.end, keys.first + sp * share), j_end = min(keys.end, keys.first + (sp + 1) * share);
 
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int li = lane % LPK, ks = lane / LPK;
@@ -103,7 +104,8 @@ attention_decode_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
         // the pages this block touches
         const int first_page = j_begin / page_size, last_page = (j_end - 1) / page_size;
         const int32_t* table = block_table + (long long)r * table_width;
-        for (int i = tid; i <= last_page - first_page && i < max_pages; i += blockDim.x) {
+        const bool gapless = keys.kept == 0;                       // with kept first positions a page is looked up key by key
+        for (int i = tid; gapless && i <= last_page - first_page && i < max_pages; i += blockDim.x) {
             const int lp = first_page + i;
             int page = lp < table_width ? table[lp] : -1;
             if (page < 0 || page >= total_pages) { *err = 3; page = -1; }
@@ -117,9 +119,15 @@ attention_decode_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
             T* vd = Vs + (size_t)stage * tile * hd;
             for (int idx = tid; idx < tile * cpr; idx += WARPS * 32) {
                 const int key = idx / cpr, c = idx % cpr;
-                const int j = j0 + key;
+                const int j = keys.at(j0 + key);
                 int page = -1;
-                if (j >= j_begin && j < j_end) page = s_table[j / page_size - first_page];
+                if (j0 + key >= j_begin && j0 + key < j_end) {
+                    if (gapless) page = s_table[j / page_size - first_page];
+                    else if (keys.visible(j)) {
+                        page = j / page_size < table_width ? table[j / page_size] : -1;
+                        if (page < 0 || page >= total_pages) { *err = 3; page = -1; }
+                    }
+                }
                 if (page >= 0) {
                     const long long off = (((long long)page * nkv + kvh) * page_size + (j % page_size)) * hd + c * EPC;
                     cp_async16(kd + key * hd + c * EPC, k_cache + off);
@@ -155,7 +163,7 @@ attention_decode_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
                 for (int u = 0; u < UNROLL; ++u) {
                     const int key = kb + ks + u * STREAMS;
                     const int j = j0 + key;
-                    ok[u] = key < tile && j >= j_begin && j < j_end;
+                    ok[u] = key < tile && j >= j_begin && j < j_end && keys.visible(keys.at(j));
 #pragma unroll
                     for (int i = 0; i < 8; ++i) { kf[u][i] = 0.f; vf[u][i] = 0.f; }
                     if (ok[u] && dim_ok) {
@@ -175,7 +183,7 @@ attention_decode_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
                         for (int i = 0; i < 8; ++i) d = fmaf(qv[g][i], kf[u][i], d);
 #pragma unroll
                         for (int o = LPK / 2; o > 0; o >>= 1) d += __shfl_xor_sync(0xffffffffu, d, o);
-                        const float far = slope[g] * (float)(p - (j0 + kb + ks + u * STREAMS));
+                        const float far = slope[g] * (float)(p - keys.at(j0 + kb + ks + u * STREAMS));
                         if (scale.softcap > 0.f) s[u] = ok[u] ? scale.softcap * tanhf((d * scale.scale) / scale.softcap) - far : -INFINITY;
                         else s[u] = ok[u] ? d * scale.scale - far : -INFINITY;
                         mx = fmaxf(mx, s[u]);

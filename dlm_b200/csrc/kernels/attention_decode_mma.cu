@@ -130,7 +130,7 @@ attention_decode_mma_kernel(const __nv_bfloat16* q, const __nv_bfloat16* k_cache
                             int table_width, const int32_t* __restrict__ cu_q, const int32_t* __restrict__ kv_len,
                             float* part_o, float* part_ml, int nh, int nkv, int page_size,
                             int page_shift, int total_pages, int window, float scale_log2, const float* __restrict__ slopes,
-                            int mask_chunk, const float* __restrict__ sinks, float cap_in, float cap_out, int chunk,
+                            int mask_chunk, const float* __restrict__ sinks, float cap_in, float cap_out, int keep, int chunk,
                             int n_splits, int head_passes, __nv_bfloat16* out, int fuse_merge, int* err) {
     constexpr int PITCH = HD + 8;
     constexpr int KS = HD / 16, DT = HD / 8, CPR = HD / 8;
@@ -153,8 +153,9 @@ attention_decode_mma_kernel(const __nv_bfloat16* q, const __nv_bfloat16* k_cache
     if (mask_chunk > 0) lo = max(lo, (p / mask_chunk) * mask_chunk);          // a chunked mask: from the chunk's start
     // the request's own visible keys, cut into n_splits equal shares (multiples of 16 keys): every split of a
     // request has the same work, whatever the longest request of the batch is
-    const int share = (((len - lo) + n_splits - 1) / n_splits + 15) & ~15;
-    const int j_begin = lo + sp * share, j_end = min(len, j_begin + share);
+    const DecodeKeys keys(lo, len, keep);       // (below, j counts keys closed up; keys.at(j) is a position)
+    const int share = (((keys.end - keys.first) + n_splits - 1) / n_splits + 15) & ~15;
+    const int j_begin = keys.first + sp * share, j_end = min(keys.end, j_begin + share);
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int t = lane & 3;
     const int token = cu_q[r];
@@ -184,15 +185,16 @@ attention_decode_mma_kernel(const __nv_bfloat16* q, const __nv_bfloat16* k_cache
             __nv_bfloat16* kd = Ks + (size_t)stage * BKV * PITCH;
             __nv_bfloat16* vd = Vs + (size_t)stage * BKV * PITCH;
             int tile_page = -1;
+            const int real0 = keys.at(j0);                        // (a tile's positions are consecutive)
             if (one_page) {
-                const int lp = j0 >> page_shift;
+                const int lp = real0 >> page_shift;
                 tile_page = lp < table_width ? table[lp] : -1;
             }
             for (int idx = tid; idx < BKV * CPR; idx += WARPS * 32) {
                 const int key = idx / CPR, c = idx % CPR;         // CPR is a compile-time constant
-                const int j = j0 + key;
+                const int j = real0 + key;
                 int page = -1, in_page = 0;
-                if (j >= j_begin && j < j_end) {
+                if (j0 + key >= j_begin && j0 + key < j_end && keys.visible(j)) {
                     if (one_page) {
                         page = tile_page;
                         in_page = j & (page_size - 1);
@@ -257,8 +259,9 @@ attention_decode_mma_kernel(const __nv_bfloat16* q, const __nv_bfloat16* k_cache
                     for (int c = 0; c < 4; ++c) {
                         const int j = jw + n * 8 + 2 * t + (c & 1);
                         // with a cap the score is cap * tanh(dot * scale / cap), in base-2 units
-                        const float far = (c < 2 ? slope_a : slope_b) * (float)(p - j);
-                        const float v = (j >= j_begin && j < j_end)
+                        const int at = keys.at(j);
+                        const float far = (c < 2 ? slope_a : slope_b) * (float)(p - at);
+                        const float v = (j >= j_begin && j < j_end && keys.visible(at))
                             ? (cap_out != 0.f ? cap_out * tanh_sfu(s[n][c] * cap_in) - far : s[n][c] * scale_log2 - far) : -INFINITY;
                         s[n][c] = v;
                         if (c < 2) mx_a = fmaxf(mx_a, v); else mx_b = fmaxf(mx_b, v);
@@ -324,6 +327,7 @@ struct DecodeTmaParams {
     int mask_chunk;
     const float* sinks;
     float cap_in, cap_out;      // cap_out != 0: a score is cap_out * tanh(dot * cap_in) (base-2 units)
+    int keep;                   // the first positions of a request, visible beyond the window
     int n_splits, head_passes;
     __nv_bfloat16* out; int fuse_merge;
     int* err;
@@ -358,8 +362,9 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
     const int len = p.kv_len[r], pos = len - 1;
     int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
     if (p.mask_chunk > 0) lo = max(lo, (pos / p.mask_chunk) * p.mask_chunk);  // a chunked mask: from the chunk's start
-    const int share = (((len - lo) + p.n_splits - 1) / p.n_splits + 15) & ~15;
-    const int j_begin = lo + sp * share, j_end = min(len, j_begin + share);
+    const DecodeKeys keys(lo, len, p.keep);     // (below, j counts keys closed up; keys.at(j) is a position)
+    const int share = (((keys.end - keys.first) + p.n_splits - 1) / p.n_splits + 15) & ~15;
+    const int j_begin = keys.first + sp * share, j_end = min(keys.end, j_begin + share);
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int t = lane & 3;
     const int token = p.cu_q[r];
@@ -381,7 +386,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
     // Everything older in the cache, the block table and the lengths were there before the step began, so the
     // producer asks for every tile that does not hold position len - 1 before it waits for that kernel;
     // everybody else waits first.
-    const int tiles_before_wait = (t_begin + n_tiles * BKV > pos) ? max(n_tiles - 1, 0) : n_tiles;
+    const int tiles_before_wait = (t_begin + n_tiles * BKV > keys.end - 1) ? max(n_tiles - 1, 0) : n_tiles;
     if (warp != WARPS) {
         dep_wait();
         dep_launch_next();
@@ -405,7 +410,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
                 // (a stage is given back only after the consumers, who have waited, have read it)
                 if (it >= tiles_before_wait && !waited) { dep_wait(); waited = true; }
                 if (it >= NST && !mbar_wait(&empty_bar[s], ((it / NST) & 1) ^ 1, abort_flag)) break;
-                const int key0 = t_begin + it * BKV;
+                const int key0 = keys.at(t_begin + it * BKV);
                 const int lp = key0 >> p.page_shift;
                 int page = lp < p.table_width ? table[lp] : -1;
                 if (page < 0 || page >= p.total_pages) { *p.err = 3; page = -1; }       // the tile holds keys of this block's share
@@ -463,8 +468,9 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
 #pragma unroll
                     for (int c = 0; c < 4; ++c) {
                         const int j = jw + n * 8 + 2 * t + (c & 1);
-                        const float far = (c < 2 ? slope_a : slope_b) * (float)(pos - j);
-                        const float v = (j >= j_begin && j < j_end)
+                        const int at = keys.at(j);
+                        const float far = (c < 2 ? slope_a : slope_b) * (float)(pos - at);
+                        const float v = (j >= j_begin && j < j_end && keys.visible(at))
                             ? (p.cap_out != 0.f ? p.cap_out * tanh_sfu(sc[n][c] * p.cap_in) - far : sc[n][c] * p.scale_log2 - far) : -INFINITY;
                         sc[n][c] = v;
                         if (c < 2) mx_a = fmaxf(mx_a, v); else mx_b = fmaxf(mx_b, v);
@@ -560,7 +566,7 @@ void launch(dim3 grid, cudaStream_t stream, const void* q, const void* k_cache, 
         static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(k_cache),
         static_cast<const __nv_bfloat16*>(v_cache), block_table, table_width, cu_q, kv_len, part_o, part_ml, nh, nkv,
         page_size, shift, total_pages, window, scale.scale * 1.4426950408889634f, scale.slopes, scale.chunk, scale.sinks,
-        scale.cap_in(), scale.cap_out(), chunk, n_splits,
+        scale.cap_in(), scale.cap_out(), scale.keep, chunk, n_splits,
         head_passes, static_cast<__nv_bfloat16*>(out), fuse_merge, error_flag_ptr());
 }
 
@@ -597,7 +603,7 @@ void attention_decode_mma(const void* q, const void* k_cache, const void* v_cach
         const dim3 tma_grid(R, nkv * head_passes, splits);
         DecodeTmaParams p{static_cast<const __nv_bfloat16*>(q), block_table, table_width, cu_q, kv_len, part_o, part_ml, nh,
                           nkv, page_size, shift, total_pages, window, scale.scale * 1.4426950408889634f, scale.slopes, scale.chunk,
-                          scale.sinks, scale.cap_in(), scale.cap_out(), splits, head_passes,
+                          scale.sinks, scale.cap_in(), scale.cap_out(), scale.keep, splits, head_passes,
                           static_cast<__nv_bfloat16*>(out), fuse_merge, error_flag_ptr()};
         // Blocks that have a multiprocessor to themselves keep six tiles in flight instead of three (8 requests
         // of 8,192 tokens: 4.72 -> 4.57 ms a step; of 1,030: 3.245 -> 3.235).

@@ -14,15 +14,19 @@ namespace dlmk {
 // logit without key or value that is not scaled.
 // softcap c > 0: the scaled dot product is squashed, c * tanh(dot * scale / c), before the distance term and the
 // mask; 0: it is used as it is.
+// keep > 0 (with a window): the first `keep` positions of the request stay visible beyond the window.
+// parts 2: query head h of the call is zero outside half h % 2 of its stored entries (two score maps share a stored
+// key side by side), so a kernel may leave the other half out of the dot product; 1: nothing is known.
 struct Score {
     float scale;
     const float* slopes;
     int chunk;
     const float* sinks;
     float softcap;
-    Score(float s, const float* b = nullptr, int c = 0, const float* k = nullptr, float cap = 0.f)
-        : scale(s), slopes(b), chunk(c), sinks(k), softcap(cap) {}
-    bool plain_mask() const { return chunk <= 0 && sinks == nullptr; }
+    int keep, parts;
+    Score(float s, const float* b = nullptr, int c = 0, const float* k = nullptr, float cap = 0.f, int kept = 0, int np = 1)
+        : scale(s), slopes(b), chunk(c), sinks(k), softcap(cap), keep(kept), parts(np) {}
+    bool plain_mask() const { return chunk <= 0 && sinks == nullptr && keep <= 0; }
     // what the tensor-core kernels get: a squashed score in base-2 units is cap_out() * tanh(dot * cap_in())
     float cap_in() const { return softcap > 0.f ? scale / softcap : 0.f; }
     float cap_out() const { return softcap > 0.f ? softcap * 1.4426950408889634f : 0.f; }
@@ -36,6 +40,38 @@ __device__ __forceinline__ float tanh_sfu(float x) {
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(x * 2.8853900817779268f));
     return 1.0f - __fdividef(2.0f, e + 1.0f);
 }
+
+// The tiles of B keys (aligned to B) that a run of queries walks when its first query's window begins at `lo` and its
+// last query is at `hi`: the tiles of the first `keep` positions as far as they end before the window's own tiles
+// begin, then the window's.
+template <int B>
+struct KeyTiles {
+    int kept, begin, n;
+    __device__ __forceinline__ KeyTiles(int lo, int hi, int keep) {
+        begin = (lo / B) * B;
+        kept = min((min(keep, lo) + B - 1) / B, begin / B);
+        n = kept + (hi - begin) / B + 1;
+    }
+    __device__ __forceinline__ int at(int it) const { return it < kept ? it * B : begin + (it - kept) * B; }
+};
+
+// The keys one decoded token sees, for kernels that cut them into shares: [0, keep) and [lo, len).  Whole blocks of
+// 64 positions between the two are left out of the count ("closed up"): index c in [first, end) stands for position
+// at(c), blocks of 64 stay blocks of 64, and every such block holds a visible key.
+struct DecodeKeys {
+    int lo, kept, first, end, gap, skip;
+    __device__ __forceinline__ DecodeKeys(int lo_, int len, int keep) {
+        lo = lo_;
+        kept = min(keep, lo);
+        const int a = (kept + 63) & ~63, b = lo & ~63;
+        skip = kept > 0 && b > a ? b - a : 0;
+        gap = skip > 0 ? a : 0x7fffffff;
+        first = kept > 0 ? 0 : lo;
+        end = len - skip;
+    }
+    __device__ __forceinline__ int at(int c) const { return c >= gap ? c + skip : c; }
+    __device__ __forceinline__ bool visible(int j) const { return j >= lo || j < kept; }
+};
 #endif
 
 // Which of the faster kernels take a chunked mask or a sink: the warp-level prefill kernel and every decode kernel

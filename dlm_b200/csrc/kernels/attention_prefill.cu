@@ -28,14 +28,15 @@ __device__ __forceinline__ float ex2(float x) {
     return y;
 }
 
-template <int HD>
+// HALVES: query head h is zero outside half h % 2 of its HD entries; the other half is left out of S = Q K^T.
+template <int HD, bool HALVES>
 __global__ void __launch_bounds__(THREADS, 2)
 attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_cache,
                          const __nv_bfloat16* __restrict__ v_cache, const int32_t* __restrict__ block_table,
                          int table_width, const int32_t* __restrict__ cu_q, const int32_t* __restrict__ kv_len,
                          __nv_bfloat16* __restrict__ out, int R, int nh, int nkv, int page_size, int total_pages,
                          int page_shift, int window, float scale_log2_arg, const float* __restrict__ slopes, int mask_chunk,
-                         const float* __restrict__ sinks, float cap_in, float cap_out, int skip_single, int n_sm,
+                         const float* __restrict__ sinks, float cap_in, float cap_out, int keep, int skip_single, int n_sm,
                          int* err) {
     constexpr int PITCH = HD + 8;              // elements per shared-memory row (16 bytes of padding)
     constexpr int KS = HD / 16;                // k16 steps over the head dimension
@@ -95,8 +96,8 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
     const int hi = pos0 + n_q - 1;
     int lo = window > 0 ? max(0, pos0 - window + 1) : 0;
     if (mask_chunk > 0) lo = max(lo, (pos0 / mask_chunk) * mask_chunk);     // the first query's chunk starts lowest
-    const int t_begin = (lo / BKV) * BKV;
-    const int n_tiles = (hi - t_begin) / BKV + 1;
+    const KeyTiles<BKV> tiles(lo, hi, keep);
+    const int n_tiles = tiles.n;
     // a tile lies within one page when pages are a power of two of at least a tile (tiles are aligned)
     const bool one_page = page_shift >= 0 && page_size >= BKV;
 
@@ -112,7 +113,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
             const int key = idx / CPR, c = idx % CPR;
             const int j = j0 + key;
             int page = -1, in_page = 0;
-            if (j >= lo && j <= hi) {
+            if ((j >= lo || j < keep) && j <= hi) {
                 if (one_page) {
                     page = tile_page;
                     in_page = j & (page_size - 1);
@@ -134,7 +135,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    fill(0, t_begin);
+    fill(0, tiles.at(0));
 
     const int g = lane >> 2, t = lane & 3;
     const int lm_row = lane & 15, lm_col = (lane >> 4) * 8;
@@ -156,9 +157,9 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
 
     for (int it = 0; it < n_tiles; ++it) {
         const int stage = it & 1;
-        const int j0 = t_begin + it * BKV;
+        const int j0 = tiles.at(it);
         if (it + 1 < n_tiles) {
-            fill(stage ^ 1, j0 + BKV);
+            fill(stage ^ 1, tiles.at(it + 1));
             asm volatile("cp.async.wait_group 1;" ::: "memory");
         } else {
             asm volatile("cp.async.wait_group 0;" ::: "memory");
@@ -167,7 +168,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
         const __nv_bfloat16* kt = Ks + (size_t)stage * BKV * PITCH;
         const __nv_bfloat16* vt = Vs + (size_t)stage * BKV * PITCH;
         // does any row of this warp see any key of the tile?
-        const bool seen = warp_live && j0 <= w_hi && (window <= 0 || j0 + BKV - 1 > w_lo - window) && j0 + BKV - 1 >= wc_lo;
+        const bool seen = warp_live && j0 <= w_hi && (window <= 0 || j0 + BKV - 1 > w_lo - window || j0 < keep) && j0 + BKV - 1 >= wc_lo;
         if (seen) {
             // S = Q K^T for 16 rows x 64 keys
             float s[BKV / 8][4];
@@ -176,7 +177,8 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
 #pragma unroll
                 for (int c = 0; c < 4; ++c) s[j][c] = 0.f;
 #pragma unroll
-            for (int kk = 0; kk < KS; ++kk) {
+            for (int k2 = 0; k2 < (HALVES ? KS / 2 : KS); ++k2) {
+                const int kk = HALVES ? k2 + (head & 1) * (KS / 2) : k2;
                 uint32_t qf[4];
                 ldsm_x4(qf, q_frag + kk * 16);
 #pragma unroll
@@ -197,7 +199,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
             const float scale_log2 = cap_out != 0.f ? 1.0f : scale_log2_arg;
             // scale (to base 2), mask where needed, running maximum
             float mx_a = m_a, mx_b = m_b;
-            const bool all_visible = j0 + BKV - 1 <= w_lo && (window <= 0 || w_hi - j0 < window) && j0 >= wc_hi;
+            const bool all_visible = j0 + BKV - 1 <= w_lo && (window <= 0 || w_hi - j0 < window || j0 + BKV - 1 < keep) && j0 >= wc_hi;
             // the distance term slope * (key - p) of an entry: a part per row and tile, a part per column of the tile
             const float far_a = slope2 * (float)(j0 + 2 * t - pa), far_b = slope2 * (float)(j0 + 2 * t - pb);
             if (all_visible && slope2 == 0.f) {
@@ -227,7 +229,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
                     for (int c = 0; c < 4; ++c) {
                         const int key = j0 + j * 8 + 2 * t + (c & 1);
                         const int p = (c < 2) ? pa : pb;
-                        const bool vis = key <= p && (window <= 0 || p - key < window) && key >= ((c < 2) ? c_a : c_b);
+                        const bool vis = key <= p && (window <= 0 || p - key < window || key < keep) && key >= ((c < 2) ? c_a : c_b);
                         const float v = vis ? fmaf(s[j][c], scale_log2, fmaf(slope2, (float)(j * 8 + (c & 1)), c < 2 ? far_a : far_b))
                                             : -INFINITY;
                         s[j][c] = v;
@@ -308,21 +310,26 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
     }
 }
 
-template <int HD>
+template <int HD, bool HALVES = false>
 void launch(dim3 grid, cudaStream_t stream, const void* q, const void* k_cache, const void* v_cache,
             const int32_t* block_table, int table_width, const int32_t* cu_q, const int32_t* kv_len, void* out, int R,
             int nh, int nkv, int page_size, int total_pages, int window, Score scale, int skip_single) {
     const size_t smem = (size_t)(BQ + 4 * BKV) * (HD + 8) * sizeof(__nv_bfloat16);
     int shift = -1;
     if ((page_size & (page_size - 1)) == 0) { shift = 0; while ((1 << shift) < page_size) ++shift; }
-    auto kern = attention_prefill_kernel<HD>;
+    if (!HALVES && HD % 32 == 0 && scale.parts == 2) {
+        launch<HD, HD % 32 == 0>(grid, stream, q, k_cache, v_cache, block_table, table_width, cu_q, kv_len, out, R, nh, nkv,
+                                 page_size, total_pages, window, scale, skip_single);
+        return;
+    }
+    auto kern = attention_prefill_kernel<HD, HALVES>;
     cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     kern<<<grid, THREADS, smem, stream>>>(
         static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(k_cache),
         static_cast<const __nv_bfloat16*>(v_cache), block_table, table_width, cu_q, kv_len,
         static_cast<__nv_bfloat16*>(out), R, nh, nkv, page_size, total_pages, shift, window,
         scale.scale * 1.4426950408889634f, scale.slopes, scale.chunk, scale.sinks, scale.cap_in(), scale.cap_out(),
-        skip_single, sm_count(), error_flag_ptr());
+        scale.keep, skip_single, sm_count(), error_flag_ptr());
 }
 
 }  // namespace

@@ -48,6 +48,8 @@ struct PrefillTcParams {
     float scale_log2;
     float cap_in, cap_out;      // cap_out != 0: a score is cap_out * tanh(dot * cap_in), in base-2 units (a cap on the scores)
     const float* sinks;         // f32 [nh] or nullptr: a logit per head in the softmax's denominator
+    int keep;                   // the first positions of a request, visible beyond the window
+    int parts;                  // 2: query head h is zero outside half h % 2 of its entries; only that half is fetched
     int skip_single;
     int* err;
 };
@@ -174,8 +176,10 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     const int pos0 = len - q_len + q0;
     const int hi = pos0 + n_q - 1;
     const int lo = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
-    const int t_begin = (lo / BKV) * BKV;
-    const int n_tiles = (hi - t_begin) / BKV + 1;
+    const KeyTiles<BKV> tiles_of(lo, hi, p.keep);
+    const int n_tiles = tiles_of.n;
+    // halves of the head dimension that enter the scores
+    const int half_lo = p.parts == 2 ? (head & 1) : 0, half_hi = p.parts == 2 ? half_lo + 1 : 2;
 
     if (warp == KEY_WARP || warp == VALUE_WARP) {
         // one warp brings the queries and the keys, another the values: a key stage is free as soon as its scores
@@ -190,15 +194,16 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             uint64_t* empty = keys ? s_full : pv_done;
             unsigned char* tiles = keys ? Ks : Vs;
             if (keys) {
-                mbar_expect_tx(&q_full, TILE_BYTES);
-                tma_load_2d(Qs, &map_q, head * HD, q_begin + q0, &q_full);
-                tma_load_2d(Qs + HALF_BYTES, &map_q, head * HD + 64, q_begin + q0, &q_full);
+                mbar_expect_tx(&q_full, (half_hi - half_lo) * HALF_BYTES);
+                for (int hf = half_lo; hf < half_hi; ++hf)
+                    tma_load_2d(Qs + hf * HALF_BYTES, &map_q, head * HD + 64 * hf, q_begin + q0, &q_full);
             }
             for (int j = 0; j < n_tiles; ++j) {
                 const int s = j & 1;
                 if (j >= 2 && !mbar_wait(&empty[s], ((j >> 1) & 1) ^ 1, abort_flag)) break;
-                mbar_expect_tx(&full[s], TILE_BYTES);
-                const int j0 = t_begin + j * BKV;
+                const int h0 = keys ? half_lo : 0, h1 = keys ? half_hi : 2;
+                mbar_expect_tx(&full[s], (h1 - h0) * HALF_BYTES);
+                const int j0 = tiles_of.at(j);
 #pragma unroll
                 for (int part = 0; part < 2; ++part) {               // two runs of 64 keys
                     const int key0 = j0 + 64 * part;
@@ -206,12 +211,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                     int page = lp < p.table_width ? table[lp] : -1;
                     if (page >= p.total_pages) page = -1;
                     // some query of the tile sees keys of this run: its page must be there
-                    if (page < 0 && key0 <= hi && key0 + 63 >= lo) *p.err = 3;
+                    if (page < 0 && key0 <= hi && (key0 + 63 >= lo || key0 < p.keep)) *p.err = 3;
                     // a run without a page is read from outside the tensor: zeros
                     const int y = page >= 0 ? (page * p.nkv + kvh) * p.page_size + (key0 & (p.page_size - 1)) : rows_total;
                     unsigned char* dst = tiles + (size_t)s * TILE_BYTES + part * (64 * 128);
-                    tma_load_2d(dst, map, 0, y, &full[s]);
-                    tma_load_2d(dst + HALF_BYTES, map, 64, y, &full[s]);
+                    for (int hf = h0; hf < h1; ++hf) tma_load_2d(dst + hf * HALF_BYTES, map, 64 * hf, y, &full[s]);
                 }
             }
         }
@@ -232,8 +236,9 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 const uint32_t d_tmem = tmem_base + (uint32_t)(j & 1) * BKV;
 #pragma unroll
                 for (int kk = 0; kk < HD / 16; ++kk) {
+                    if ((kk >> 2) < half_lo || (kk >> 2) >= half_hi) continue;
                     const uint64_t off = (uint64_t)((kk >> 2) * (HALF_BYTES >> 4) + (kk & 3) * 2);
-                    umma_bf16(d_tmem, dq + off, dkj + off, IDESC_S, kk > 0 ? 1u : 0u);
+                    umma_bf16(d_tmem, dq + off, dkj + off, IDESC_S, kk > half_lo * 4 ? 1u : 0u);
                 }
                 umma_commit(&s_full[j & 1]);         // the scores are there, and the keys of the stage are read
             };
@@ -282,7 +287,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         float m = -INFINITY, l = 0.f;
         bool ok = true;
         for (int j = 0; j < n_tiles; ++j) {
-            const int j0 = t_begin + j * BKV;
+            const int j0 = tiles_of.at(j);
             const uint32_t s_tmem = tmem_base + (uint32_t)(j & 1) * BKV + lane_base;
             // (the outcome of a wait is made the same for the whole warp: the collectives below need all lanes)
             if (!__all_sync(0xffffffffu, mbar_wait(&s_full[j & 1], (j >> 1) & 1, abort_flag))) { ok = false; break; }
@@ -305,7 +310,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             }
             const float sl2 = p.cap_out != 0.f ? 1.0f : p.scale_log2;
             // does every row of this warp see every key of the tile?  Then nothing is masked.
-            const bool row_all = j0 + BKV - 1 <= pos && (p.window <= 0 || pos - j0 < p.window);
+            const bool row_all = j0 + BKV - 1 <= pos && (p.window <= 0 || pos - j0 < p.window || j0 + BKV - 1 < p.keep);
             const bool warp_all = __all_sync(0xffffffffu, row_all);
             if (!warp_all) {
 #pragma unroll
@@ -313,7 +318,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 #pragma unroll
                     for (int i = 0; i < 32; ++i) {
                         const int key = j0 + c * 32 + i;
-                        const bool vis = key <= pos && (p.window <= 0 || pos - key < p.window);
+                        const bool vis = key <= pos && (p.window <= 0 || pos - key < p.window || key < p.keep);
                         if (!vis) v[c][i] = 0xff800000u;             // -inf
                     }
             }
@@ -472,7 +477,8 @@ bool attention_prefill_tc(const void* q, const void* k_cache, const void* v_cach
     int shift = 0;
     while ((1 << shift) < page_size) ++shift;
     PrefillTcParams p{block_table, table_width, cu_q, kv_len, static_cast<__nv_bfloat16*>(out), R, nh, nkv, page_size,
-                      shift, total_pages, window, scale.scale * 1.4426950408889634f, scale.cap_in(), scale.cap_out(), scale.sinks, skip_single,
+                      shift, total_pages, window, scale.scale * 1.4426950408889634f, scale.cap_in(), scale.cap_out(), scale.sinks,
+                      scale.keep, scale.parts, skip_single,
                       error_flag_ptr()};
     const size_t smem = (size_t)TILE_BYTES * 7 + 1024;      // Q, 2 x K, 2 x V, 2 x P, and room to align
     cudaFuncSetAttribute(attention_prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);

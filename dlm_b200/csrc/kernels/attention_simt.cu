@@ -82,17 +82,21 @@ attention_simt_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, co
     int lo = 0;
     if (window > 0) lo = max(0, pos0 - window + 1);
     if (scale.chunk > 0) lo = max(lo, (pos0 / scale.chunk) * scale.chunk);   // the first query's chunk starts lowest
-    const int tile_lo = (lo / BKV) * BKV;
+    const int keep = scale.keep;                    // the first positions, visible beyond the window
+    const KeyTiles<BKV> tiles(lo, hi, keep);
     const int* table = block_table + (long long)r * table_width;
+    // the entries of the head that can differ from zero
+    const int d_lo = scale.parts == 2 ? (head & 1) * (hd / 2) : 0, d_hi = scale.parts == 2 ? d_lo + hd / 2 : hd;
 
-    for (int kv0 = tile_lo; kv0 <= hi; kv0 += BKV) {
+    for (int it = 0; it < tiles.n; ++it) {
+        const int kv0 = tiles.at(it);
         __syncthreads();
         // load the tile: key j = kv0 + jj
         for (int idx = tid; idx < BKV * hd; idx += blockDim.x) {
             const int jj = idx / hd, d = idx % hd;
             const int j = kv0 + jj;
             float kvv = 0.f, vvv = 0.f;
-            if (j <= hi && j >= lo) {
+            if (j <= hi && (j >= lo || j < keep)) {
                 const int lp = j / page_size;
                 const int page = lp < table_width ? table[lp] : -1;
                 if (page >= 0 && page < total_pages) {
@@ -117,10 +121,10 @@ attention_simt_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, co
             const float* qv = Qs + qi * hd;
             const float* kr = Ks + lane * (hd + 1);
             float s = 0.f;
-            for (int d = 0; d < hd; ++d) s = fmaf(qv[d], kr[d], s);
+            for (int d = d_lo; d < d_hi; ++d) s = fmaf(qv[d], kr[d], s);
             if (scale.softcap > 0.f) s = scale.softcap * tanhf((s * scale.scale) / scale.softcap) - slope * (float)(p - j);
             else s = s * scale.scale - slope * (float)(p - j);
-            const bool visible = (j <= p) && (window <= 0 || p - j < window) &&
+            const bool visible = (j <= p) && (window <= 0 || p - j < window || j < keep) &&
                                  (scale.chunk <= 0 || j >= (p / scale.chunk) * scale.chunk);
             if (!visible) s = -INFINITY;
             const float m_new = fmaxf(m[i], warp_max(s));

@@ -20,6 +20,7 @@ PYBIND11_MODULE(_dlm_kernels, m) {
     m.attr("EPI_GELU") = (int)dlmk::EPI_GELU;
     m.attr("EPI_GELU_TANH") = (int)dlmk::EPI_GELU_TANH;
     m.attr("EPI_GEGLU_TANH") = (int)dlmk::EPI_GEGLU_TANH;
+    m.attr("EPI_CLAMP_GLU") = (int)dlmk::EPI_CLAMP_GLU;
 
     m.def("embed", [](u64 tokens, u64 table, u64 out, int T, int H, int V, float scale, int dtype, u64 stream) {
         dlmk::embed(ptr<const int32_t>(tokens), ptr<const void>(table), ptr<float>(out), T, H, V, scale, dtype,
@@ -45,13 +46,13 @@ PYBIND11_MODULE(_dlm_kernels, m) {
     });
     m.def("attention", [](u64 q, u64 k_cache, u64 v_cache, u64 block_table, int table_width, u64 cu_q, u64 kv_len,
                           u64 out, int T, int R, int nh, int nkv, int hd, int page_size, int total_pages, int window,
-                          float scale, u64 slopes, int chunk, u64 sinks, float softcap, int max_q_len, int max_kv_len,
-                          int num_single, u64 scratch, int dtype, int fast, u64 stream) {
+                          float scale, u64 slopes, int chunk, u64 sinks, float softcap, int keep, int parts, int max_q_len,
+                          int max_kv_len, int num_single, u64 scratch, int dtype, int fast, u64 stream) {
         dlmk::attention(ptr<const void>(q), ptr<const void>(k_cache), ptr<const void>(v_cache),
                         ptr<const int32_t>(block_table), table_width, ptr<const int32_t>(cu_q),
                         ptr<const int32_t>(kv_len), ptr<void>(out), T, R, nh, nkv, hd, page_size, total_pages, window,
-                        scale, ptr<const float>(slopes), chunk, ptr<const float>(sinks), softcap, max_q_len, max_kv_len,
-                        num_single, ptr<float>(scratch), dtype, fast, st(stream));
+                        scale, ptr<const float>(slopes), chunk, ptr<const float>(sinks), softcap, keep, parts, max_q_len,
+                        max_kv_len, num_single, ptr<float>(scratch), dtype, fast, st(stream));
     });
     m.def("attention_scratch_floats", [](int R, int nh, int nkv, int hd, int max_kv_len) {
         return dlmk::attention_scratch_floats(R, nh, nkv, hd, max_kv_len);
@@ -266,6 +267,25 @@ PYBIND11_MODULE(_dlm_kernels, m) {
                             T, H, out_dtype, st(stream));
     });
     m.def("tanh_cap", [](u64 x, long long n, float cap, u64 stream) { dlmk::tanh_cap(ptr<float>(x), n, cap, st(stream)); });
+    m.def("map_norm_write", [](u64 proj, int ld, u64 conv, int taps, u64 state, u64 cu_q, u64 token_req, u64 state_slot,
+                               u64 qn, u64 kn, float eps, u64 slots, u64 q_out, u64 k_cache, u64 v_cache, int T, int R,
+                               int num_single, int H, int G, int d, int dv, int D, int page_size, int total_pages,
+                               int dtype, u64 stream) {
+        dlmk::map_norm_write(ptr<const float>(proj), ld, ptr<const float>(conv), taps, ptr<float>(state),
+                             ptr<const int32_t>(cu_q), ptr<const int32_t>(token_req), ptr<const int32_t>(state_slot),
+                             ptr<const float>(qn), ptr<const float>(kn), eps, ptr<const int32_t>(slots), ptr<void>(q_out),
+                             ptr<void>(k_cache), ptr<void>(v_cache), T, R, num_single, H, G, d, dv, D, page_size,
+                             total_pages, dtype, st(stream));
+    });
+    m.def("diff_norm_gate", [](u64 o, u64 gate, int ldg, u64 out, int T, int H, int dv, int D, float lambda, float eps,
+                               float factor, int dtype, u64 stream) {
+        dlmk::diff_norm_gate(ptr<const void>(o), ptr<const float>(gate), ldg, ptr<void>(out), T, H, dv, D, lambda, eps,
+                             factor, dtype, st(stream));
+    });
+    m.def("weigh_rows", [](u64 h, u64 wts, u64 dest, u64 out, int T, int k, int H, int dtype, u64 stream) {
+        dlmk::weigh_rows(ptr<const void>(h), ptr<const float>(wts), ptr<const int32_t>(dest), ptr<void>(out), T, k, H,
+                         dtype, st(stream));
+    });
     m.def("entry_gate", [](u64 o, u64 gate, int ldg, int T, int nh, int dv, int D, float factor, int dtype, u64 resid,
                            u64 bias, int W, u64 stream) {
         dlmk::entry_gate(ptr<void>(o), ptr<const float>(gate), ldg, T, nh, dv, D, factor, dtype, ptr<float>(resid),

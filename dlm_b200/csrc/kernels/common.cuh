@@ -107,14 +107,24 @@ __device__ __forceinline__ float gelu_tanh_f(float z) {
 template <int EPI> __device__ __forceinline__ float epi_act(float v) {
     return EPI == 3 ? gelu_exact_f(v) : (EPI == 4 ? gelu_tanh_f(v) : v);
 }
-// The gated epilogues, 2 (EPI_SWIGLU) and 5 (EPI_GEGLU_TANH): what the gate half goes through before it meets the up
+// The gated epilogues, 2 (EPI_SWIGLU), 5 (EPI_GEGLU_TANH) and 6 (EPI_CLAMP_GLU): what the gate half goes through before it meets the up
 // half.  glu_act_fast: for results that are rounded to bfloat16 (fast exponential and division; the tanh form of gelu
 // is z times the logistic function of twice the tanh's argument).
-constexpr bool epi_is_glu(int epi) { return epi == 2 || epi == 5; }
+constexpr bool epi_is_glu(int epi) { return epi == 2 || epi == 5 || epi == 6; }
+// whether the `bias` of a product is something the epilogue may read (a bias, or the constants of EPI_CLAMP_GLU)
+constexpr bool epi_takes_bias(int epi) { return epi == 0 || epi == 3 || epi == 4 || epi == 6; }
 template <int EPI> __device__ __forceinline__ float glu_act(float g) { return EPI == 5 ? gelu_tanh_f(g) : silu_f(g); }
 template <int EPI> __device__ __forceinline__ float glu_act_fast(float g) {
     const float z = EPI == 5 ? 1.59576912160573071176f * (g + 0.044715f * g * g * g) : g;
     return __fdividef(g, 1.0f + __expf(-z));
+}
+// One output of a gated epilogue from its gate and up sums; `c`: the constants of EPI_CLAMP_GLU {limit, alpha, shift}.
+template <int EPI, bool FAST> __device__ __forceinline__ float glu_out(float g, float u, const float* c) {
+    if (EPI == 6) {
+        const float limit = c[0], z = fminf(g, limit), v = fminf(fmaxf(u, -limit), limit) + c[2];
+        return (FAST ? __fdividef(z, 1.0f + __expf(-c[1] * z)) : z / (1.0f + expf(-c[1] * z))) * v;
+    }
+    return (FAST ? glu_act_fast<EPI>(g) : glu_act<EPI>(g)) * u;
 }
 
 }  // namespace dlmk

@@ -362,7 +362,7 @@ __global__ void moe_combine_kernel(const float* y, const int32_t* dest,
         for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < H / 4; i += blockDim.x * gridDim.y) {
             float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
             for (int j = 0; j < k; ++j) {
-                const float wj = wts[t * k + j];
+                const float wj = wts != nullptr ? wts[t * k + j] : 1.0f;
                 const float4 v = *reinterpret_cast<const float4*>(source(j) + 4 * i);
                 acc.x = fmaf(wj, v.x, acc.x); acc.y = fmaf(wj, v.y, acc.y);
                 acc.z = fmaf(wj, v.z, acc.z); acc.w = fmaf(wj, v.w, acc.w);
@@ -380,7 +380,7 @@ __global__ void moe_combine_kernel(const float* y, const int32_t* dest,
         for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < H; i += blockDim.x * gridDim.y) {
             float acc = 0.f;
             for (int j = 0; j < k; ++j)
-                acc = fmaf(wts[t * k + j], source(j)[i], acc);
+                acc = fmaf(wts != nullptr ? wts[t * k + j] : 1.0f, source(j)[i], acc);
             if (shared != nullptr) {
                 const float g = (gate ? gate[t] : 1.0f) * shared_scale;
                 acc = fmaf(g, shared[(long long)t * H + i], acc);

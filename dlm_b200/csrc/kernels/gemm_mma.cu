@@ -167,7 +167,7 @@ __global__ void __launch_bounds__(THREADS) gemm_mma_kernel(MmaParams p) {
                 const float v0 = acc[i][j][half * 2], v1 = acc[i][j][half * 2 + 1];
                 if (epi_is_glu(EPI)) {
                     if (col + 1 < p.N)
-                        static_cast<TOut*>(p.out)[(long long)row * p.ldo + (col >> 1)] = from_f32<TOut>(glu_act<EPI>(v0) * v1);
+                        static_cast<TOut*>(p.out)[(long long)row * p.ldo + (col >> 1)] = from_f32<TOut>(glu_out<EPI, false>(v0, v1, p.bias));
                 } else if (EPI == EPI_ADD) {
                     float* o = static_cast<float*>(p.out) + (long long)row * p.ldo;
                     if (col < p.N) o[col] += v0;
@@ -196,6 +196,7 @@ void launch_bm(const MmaParams& p, int epilogue, dim3 grid, cudaStream_t stream)
         case EPI_GELU: DLM_MMA(EPI_GELU, TOut) break;
         case EPI_GELU_TANH: DLM_MMA(EPI_GELU_TANH, TOut) break;
         case EPI_GEGLU_TANH: DLM_MMA(EPI_GEGLU_TANH, TOut) break;
+        case EPI_CLAMP_GLU: DLM_MMA(EPI_CLAMP_GLU, TOut) break;
         default: DLM_MMA(EPI_SWIGLU, TOut) break;
     }
 #undef DLM_MMA
@@ -209,7 +210,8 @@ void gemm_mma(const void* a, int lda, const int32_t* a_rows, const void* w, int 
     if (M <= 0 || N <= 0) return;
     DLM_CHECK(!epi_is_glu(epilogue) || N % 2 == 0, "gemm: a gated epilogue needs an even N");
     DLM_CHECK(epilogue != EPI_ADD || out_dtype == F32, "gemm: the accumulate epilogue needs a float32 output");
-    DLM_CHECK(bias == nullptr || epilogue == EPI_STORE || epilogue == EPI_GELU || epilogue == EPI_GELU_TANH, "gemm: a bias goes with a storing epilogue only");
+    DLM_CHECK(bias == nullptr || epi_takes_bias(epilogue), "gemm: a bias goes with a storing epilogue only");
+    DLM_CHECK(epilogue != EPI_CLAMP_GLU || bias != nullptr, "gemm: the clamped gate needs its constants");
     MmaParams p{static_cast<const __nv_bfloat16*>(a), lda, a_rows, static_cast<const __nv_bfloat16*>(w), ldw,
                 w_expert_stride, expert_offsets, num_experts, bias, out, ldo, M, N, K};
     // grouped products have ragged groups: smaller row tiles waste less

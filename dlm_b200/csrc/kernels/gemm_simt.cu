@@ -109,7 +109,7 @@ __global__ void __launch_bounds__(THREADS) gemm_simt_kernel(GemmParams p) {
 #pragma unroll
             for (int j = 0; j < 4; j += 2) {
                 const int col = n0 + tx * 4 + j;
-                if (col + 1 < p.N) o[col >> 1] = from_f32<TOut>(glu_act<EPI>(acc[i][j]) * acc[i][j + 1]);
+                if (col + 1 < p.N) o[col >> 1] = from_f32<TOut>(glu_out<EPI, false>(acc[i][j], acc[i][j + 1], p.bias));
             }
         } else if (EPI == EPI_ADD) {
             float* o = static_cast<float*>(p.out) + (long long)row * p.ldo;
@@ -138,6 +138,7 @@ void launch(const GemmParams& p, int epilogue, dim3 grid, cudaStream_t stream) {
         case EPI_GELU: gemm_simt_kernel<TIn, TOut, EPI_GELU><<<grid, THREADS, 0, stream>>>(p); break;
         case EPI_GELU_TANH: gemm_simt_kernel<TIn, TOut, EPI_GELU_TANH><<<grid, THREADS, 0, stream>>>(p); break;
         case EPI_GEGLU_TANH: gemm_simt_kernel<TIn, TOut, EPI_GEGLU_TANH><<<grid, THREADS, 0, stream>>>(p); break;
+        case EPI_CLAMP_GLU: gemm_simt_kernel<TIn, TOut, EPI_CLAMP_GLU><<<grid, THREADS, 0, stream>>>(p); break;
         default: DLM_CHECK(false, "gemm: unknown epilogue");
     }
 }
@@ -151,7 +152,8 @@ void gemm_simt(const void* a, int lda, const int32_t* a_rows, const void* w, int
     DLM_CHECK(K > 0, "gemm: K must be > 0");
     DLM_CHECK(!epi_is_glu(epilogue) || N % 2 == 0, "gemm: a gated epilogue needs an even N");
     DLM_CHECK(epilogue != EPI_ADD || out_dtype == F32, "gemm: the accumulate epilogue needs a float32 output");
-    DLM_CHECK(bias == nullptr || epilogue == EPI_STORE || epilogue == EPI_GELU || epilogue == EPI_GELU_TANH, "gemm: a bias goes with a storing epilogue only");
+    DLM_CHECK(bias == nullptr || epi_takes_bias(epilogue), "gemm: a bias goes with a storing epilogue only");
+    DLM_CHECK(epilogue != EPI_CLAMP_GLU || bias != nullptr, "gemm: the clamped gate needs its constants");
     GemmParams p{a, lda, a_rows, w, ldw, w_expert_stride, expert_offsets, num_experts, bias, out, ldo, M, N, K};
     int m_tiles = (M + BM - 1) / BM;
     if (expert_offsets != nullptr) {

@@ -185,7 +185,7 @@ __global__ void __launch_bounds__(WARPS * 32) gemm_smallm_kernel(SmallParams p) 
                     up += red[rr * S + ss][2 * pr + 1][m];
                 }
                 static_cast<TOut*>(p.out)[(long long)(row0 + m0 + m) * p.ldo + (n >> 1)] =
-                    from_f32<TOut>(glu_act<EPI>(gate) * up);
+                    from_f32<TOut>(glu_out<EPI, false>(gate, up, p.bias));
             }
         } else {
             for (int i = tid; i < R * MP * 16; i += WARPS * 32) {
@@ -210,6 +210,7 @@ void launch_nt(const SmallParams& p, int epilogue, dim3 grid, cudaStream_t strea
         case EPI_GELU: launch_dep(gemm_smallm_kernel<NT, EPI_GELU, TOut>, grid, WARPS * 32, 0, stream, p); break;
         case EPI_GELU_TANH: launch_dep(gemm_smallm_kernel<NT, EPI_GELU_TANH, TOut>, grid, WARPS * 32, 0, stream, p); break;
         case EPI_GEGLU_TANH: launch_dep(gemm_smallm_kernel<NT, EPI_GEGLU_TANH, TOut>, grid, WARPS * 32, 0, stream, p); break;
+        case EPI_CLAMP_GLU: launch_dep(gemm_smallm_kernel<NT, EPI_CLAMP_GLU, TOut>, grid, WARPS * 32, 0, stream, p); break;
         default: launch_dep(gemm_smallm_kernel<NT, EPI_SWIGLU, TOut>, grid, WARPS * 32, 0, stream, p); break;
     }
 }

@@ -357,7 +357,7 @@ __global__ void __launch_bounds__(THREADS, 1) gemm_stream_kernel(StreamParams p)
                             up += rb[((size_t)ww * 16 + 2 * pr + 1) * (MP + 1) + m];
                         }
                         static_cast<TOut*>(p.out)[(long long)(out_row0 + m) * p.ldo + (n >> 1)] =
-                            from_f32<TOut>(glu_act<EPI>(gate) * up);
+                            from_f32<TOut>(glu_out<EPI, false>(gate, up, p.bias));
                     }
                 } else {
 #pragma unroll
@@ -403,6 +403,8 @@ void launch_nt(const StreamParams& p, int grid, int out_dtype, int epilogue, cud
                        else launch_one<NT, NCH, EPI_GELU_TANH, __nv_bfloat16>(p, grid, stream); break;
         case EPI_GEGLU_TANH: if (f32) launch_one<NT, NCH, EPI_GEGLU_TANH, float>(p, grid, stream);
                        else launch_one<NT, NCH, EPI_GEGLU_TANH, __nv_bfloat16>(p, grid, stream); break;
+        case EPI_CLAMP_GLU: if (f32) launch_one<NT, NCH, EPI_CLAMP_GLU, float>(p, grid, stream);
+                       else launch_one<NT, NCH, EPI_CLAMP_GLU, __nv_bfloat16>(p, grid, stream); break;
         default: if (f32) launch_one<NT, NCH, EPI_SWIGLU, float>(p, grid, stream);
                  else launch_one<NT, NCH, EPI_SWIGLU, __nv_bfloat16>(p, grid, stream); break;
     }

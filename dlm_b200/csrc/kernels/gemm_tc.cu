@@ -252,7 +252,8 @@ bool gemm_tc(const void* a, int lda, const void* w, int ldw, const int32_t* expe
     if (M <= 0 || N <= 0) return true;
     DLM_CHECK(!epi_is_glu(epilogue) || N % 2 == 0, "gemm: a gated epilogue needs an even N");
     DLM_CHECK(epilogue != EPI_ADD || out_dtype == F32, "gemm: the accumulate epilogue needs a float32 output");
-    DLM_CHECK(bias == nullptr || epilogue == EPI_STORE || epilogue == EPI_GELU || epilogue == EPI_GELU_TANH, "gemm: a bias goes with a storing epilogue only");
+    DLM_CHECK(bias == nullptr || epi_takes_bias(epilogue), "gemm: a bias goes with a storing epilogue only");
+    DLM_CHECK(epilogue != EPI_CLAMP_GLU || bias != nullptr, "gemm: the clamped gate needs its constants");
     if (N > BM && gemm_tc_pair_enabled() &&
         gemm_tc_pair(a, lda, w, ldw, expert_offsets, num_experts, bias, out, ldo, M, N, K, out_dtype, epilogue, stream))
         return true;
@@ -288,6 +289,8 @@ bool gemm_tc(const void* a, int lda, const void* w, int ldw, const int32_t* expe
                        else launch<G, EPI_GELU_TANH, __nv_bfloat16>(mw, ma, p, nx, total_tiles, stream); break;  \
         case EPI_GEGLU_TANH: if (f32) launch<G, EPI_GEGLU_TANH, float>(mw, ma, p, nx, total_tiles, stream);      \
                        else launch<G, EPI_GEGLU_TANH, __nv_bfloat16>(mw, ma, p, nx, total_tiles, stream); break; \
+        case EPI_CLAMP_GLU: if (f32) launch<G, EPI_CLAMP_GLU, float>(mw, ma, p, nx, total_tiles, stream);        \
+                       else launch<G, EPI_CLAMP_GLU, __nv_bfloat16>(mw, ma, p, nx, total_tiles, stream); break; \
         default: if (f32) launch<G, EPI_SWIGLU, float>(mw, ma, p, nx, total_tiles, stream);                 \
                  else launch<G, EPI_SWIGLU, __nv_bfloat16>(mw, ma, p, nx, total_tiles, stream); break;      \
     }

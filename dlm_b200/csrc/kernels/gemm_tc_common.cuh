@@ -86,7 +86,7 @@ __device__ __forceinline__ void epilogue_tile(const TcParams& p, float* st, uint
                 const float a0 = __uint_as_float(v[j]), a1 = __uint_as_float(v[j + 1]);
                 const float got = __shfl_xor_sync(0xffffffffu, odd ? a0 : a1, 1);
                 const float g = odd ? got : a0, uu = odd ? a1 : got;
-                st[(j + (odd ? 1 : 0)) * 17 + (lane >> 1)] = glu_act_fast<EPI>(g) * uu;
+                st[(j + (odd ? 1 : 0)) * 17 + (lane >> 1)] = glu_out<EPI, true>(g, uu, p.bias);
             }
             __syncwarp();
             TOut* o = static_cast<TOut*>(p.out) + (long long)tok0 * p.ldo + (colw >> 1);

@@ -331,6 +331,8 @@ bool gemm_tc_pair(const void* a, int lda, const void* w, int ldw, const int32_t*
                        else launch<ST, AR, EPI_GELU_TANH, __nv_bfloat16>(mw, ma, p, nx, total_tiles, tt, stream); break; \
         case EPI_GEGLU_TANH: if (f32) launch<ST, AR, EPI_GEGLU_TANH, float>(mw, ma, p, nx, total_tiles, tt, stream);   \
                        else launch<ST, AR, EPI_GEGLU_TANH, __nv_bfloat16>(mw, ma, p, nx, total_tiles, tt, stream); break; \
+        case EPI_CLAMP_GLU: if (f32) launch<ST, AR, EPI_CLAMP_GLU, float>(mw, ma, p, nx, total_tiles, tt, stream);     \
+                       else launch<ST, AR, EPI_CLAMP_GLU, __nv_bfloat16>(mw, ma, p, nx, total_tiles, tt, stream); break; \
         default: if (f32) launch<ST, AR, EPI_SWIGLU, float>(mw, ma, p, nx, total_tiles, tt, stream);              \
                  else launch<ST, AR, EPI_SWIGLU, __nv_bfloat16>(mw, ma, p, nx, total_tiles, tt, stream); break;   \
     }

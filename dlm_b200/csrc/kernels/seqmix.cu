@@ -189,11 +189,12 @@ __global__ void causal_conv_kernel(const float* __restrict__ x, int ldx, const f
 // owns a (request, channel): it reads what it needs before it writes.
 constexpr int MAX_TAPS = 16;
 __global__ void conv_state_kernel(const float* __restrict__ x, int ldx, float* state, const int32_t* __restrict__ cu_q,
-                                  const int32_t* __restrict__ state_slot, int C, int taps) {
+                                  const int32_t* __restrict__ state_slot, int C, int taps, int skip_single) {
     dep_wait();          // nothing is read or written before the kernels before this one have ended
     dep_launch_next();
     const int r = blockIdx.x;
     const int start = cu_q[r], n = cu_q[r + 1] - start;
+    if (skip_single && n == 1) return;
     const int keep = taps - 1;
     float* st = state + (long long)state_slot[r] * keep * C;
     for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < C; c += gridDim.y * blockDim.x) {
@@ -785,10 +786,15 @@ void causal_conv(const float* x, int ldx, const float* w, const float* bias, flo
             x, ldx, w, bias, state, cu_q, token_req, state_slot, C, taps, add_input, act,
             static_cast<__nv_bfloat16*>(out), ldo);
     check_launch("causal_conv");
-    if (taps > 1) {
-        launch_dep(conv_state_kernel, dim3(R, slices), dim3(256), 0, stream, x, ldx, state, cu_q, state_slot, C, taps);
-        check_launch("conv_state");
-    }
+    if (taps > 1) conv_state(x, ldx, state, cu_q, state_slot, R, C, taps, 0, stream);
+}
+
+void conv_state(const float* x, int ldx, float* state, const int32_t* cu_q, const int32_t* state_slot, int R, int C,
+                int taps, int skip_single, cudaStream_t stream) {
+    DLM_CHECK(taps >= 2 && taps <= MAX_TAPS, "conv_state: 2 to 16 taps");
+    launch_dep(conv_state_kernel, dim3(R, (C + 255) / 256), dim3(256), 0, stream, x, ldx, state, cu_q, state_slot, C, taps,
+               skip_single);
+    check_launch("conv_state");
 }
 
 void activation(const float* x, int ldx, void* out, int ldo, int rows, int cols, int op, int out_dtype,

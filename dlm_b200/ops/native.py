@@ -393,6 +393,51 @@ class NativeOps:
                                     _p(slots), _p(q), _p(k_cache), _p(v_cache), T, nh, nkv, d, dv, D, page_size, total_pages, _dt(out_dtype), self._stream())
         return q
 
+    def map_norm_write(self, proj, conv_w, state, batch, qn_w, kn_w, eps, slots, k_cache, v_cache, H, G, d, dv, D, out_dtype):
+        """Attention heads with two score maps.  ``proj`` 32-bit rows ``[q: H x 2 x d | k: G x 2 x d | v: G x dv | ...]``;
+        every channel first passes a causal convolution over time (``conv_w`` ``[taps, C]``, None: none; ``state``
+        ``[slots, taps - 1, C]`` carries each request's last inputs and is brought up to date); every map of q and k is
+        divided by its root mean square and multiplied by ``qn_w`` / ``kn_w`` ``[d]``.  Returns q ``[T, 2H * D]`` with
+        map m's query in half m of its D entries; a token's two keys fill the halves of its stored key."""
+        T = proj.shape[0]
+        C = 2 * (H + G) * d + G * dv
+        taps = conv_w.shape[0] if conv_w is not None else 1
+        assert proj.dtype == torch.float32 and proj.stride(1) == 1 and proj.shape[1] >= C
+        assert conv_w is None or (conv_w.shape[1] == C and conv_w.is_contiguous() and conv_w.dtype == torch.float32)
+        assert taps == 1 or (state.shape[1:] == (taps - 1, C) and state.dtype == torch.float32)
+        total_pages, g_c, page_size, D_c = k_cache.shape
+        assert (g_c, D_c) == (G, D) and k_cache.dtype == out_dtype and v_cache.shape == k_cache.shape
+        q = torch.empty((T, 2 * H * D), dtype=out_dtype, device=proj.device)
+        self.launches += 2 if taps > 1 and batch.num_single < batch.num_requests else 1
+        self.k.map_norm_write(_p(proj), proj.stride(0), _p(conv_w), taps, _p(state if taps > 1 else None), _p(batch.cu_q),
+                              _p(batch.token_req), _p(batch.state_slot), _p(qn_w), _p(kn_w), float(eps), _p(slots), _p(q),
+                              _p(k_cache), _p(v_cache), T, batch.num_requests, int(batch.num_single), H, G, d, dv, D,
+                              page_size, total_pages, _dt(out_dtype), self._stream())
+        return q
+
+    def diff_norm_gate(self, o, gate, H, dv, D, lam, eps, factor):
+        """``c = o[:, 2h] - lam * o[:, 2h + 1]`` over the first ``dv`` of D entries, divided by its root mean square,
+        times ``factor * sigmoid(gate)`` (``gate`` 32-bit raw ``[T, H * dv]``, may be a column slice; None: no gate).
+        Returns ``[T, H * dv]`` in ``o``'s dtype."""
+        T = o.shape[0]
+        assert o.shape[1] == 2 * H * D and o.is_contiguous()
+        assert gate is None or (gate.dtype == torch.float32 and gate.shape == (T, H * dv) and gate.stride(1) == 1)
+        out = torch.empty((T, H * dv), dtype=o.dtype, device=o.device)
+        self.launches += 1
+        self.k.diff_norm_gate(_p(o), _p(gate), 0 if gate is None else gate.stride(0), _p(out), T, H, dv, D, float(lam),
+                              float(eps), float(factor), _dt(o.dtype), self._stream())
+        return out
+
+    def weigh_rows(self, h, wts, dest):
+        """``out[dest[t, j]] = wts[t, j] * h[t]``: the rows of every expert side by side, each already weighted."""
+        T, H = h.shape
+        k = dest.shape[1]
+        assert h.is_contiguous() and wts.shape == (T, k) and dest.shape == (T, k)
+        out = torch.empty((T * k, H), dtype=h.dtype, device=h.device)
+        self.launches += 1
+        self.k.weigh_rows(_p(h), _p(wts), _p(dest), _p(out), T, k, H, _dt(h.dtype), self._stream())
+        return out
+
     def head_gate(self, o, gate, nh, D, factor=1.0):
         """``o[t, h * D + i] *= factor * sigmoid(gate[t, h])`` in place (``gate`` 32-bit, may be a column slice)."""
         T = o.shape[0]
@@ -609,8 +654,24 @@ class NativeOps:
         self._gemm(a, w_gate_up, out, M, N, K, epi)
         return out
 
+    def linear_clamped_glu(self, a, w_gate_up, constants):
+        """``g sigmoid(alpha g) (u + shift)`` of a product with interleaved gate and up rows, g at most ``limit`` and u
+        within ``+-limit``, as an epilogue; ``constants``: 32-bit ``[limit, alpha, shift]`` on the device."""
+        (M, K), N = a.shape, w_gate_up.shape[0]
+        assert w_gate_up.shape[1] == K and a.dtype == w_gate_up.dtype
+        assert constants.shape == (3,) and constants.dtype == torch.float32
+        out = torch.empty((M, N // 2), dtype=a.dtype, device=a.device)
+        self._gemm(a, w_gate_up, out, M, N, K, self.k.EPI_CLAMP_GLU, bias=constants)
+        return out
+
     def grouped_swiglu(self, a, w_gate_up, offsets, rows):
+        """``rows`` None: the rows of ``a`` are already grouped by expert."""
         E, N, K = w_gate_up.shape
+        if rows is None:
+            out = torch.empty((a.shape[0], N // 2), dtype=a.dtype, device=a.device)
+            self._gemm(a, w_gate_up, out, a.shape[0], N, K, self.k.EPI_SWIGLU, offsets=offsets, num_experts=E,
+                       w_expert_stride=N * K)
+            return out
         M = rows.numel()
         out = torch.empty((M, N // 2), dtype=a.dtype, device=a.device)
         if (self.fast and self.tc and a.dtype == torch.bfloat16 and 8 * M > 9 * E and K % 8 == 0
@@ -680,11 +741,12 @@ class NativeOps:
         return q
 
     def attention(self, q, k_cache, v_cache, block_table, cu_q, kv_len, window, scale, nh, nkv, hd, max_q_len,
-                  max_kv_len, num_single=0, slopes=None, chunk=0, sinks=None, softcap=0.0):
+                  max_kv_len, num_single=0, slopes=None, chunk=0, sinks=None, softcap=0.0, keep_first=0, parts=1):
         """``slopes`` (32-bit ``[nh]`` or None): a score loses ``slopes[head] * (query position - key position)``.
         ``chunk`` > 0: a query at p sees only keys from ``floor(p / chunk) * chunk`` on.  ``sinks`` (32-bit ``[nh]`` or
         None): the softmax's denominator also holds ``exp(sinks[head])``.  ``softcap`` c > 0: the scaled dot product
-        becomes ``c tanh(. / c)`` first."""
+        becomes ``c tanh(. / c)`` first.  ``keep_first`` with a window: the first positions of a request stay visible.
+        ``parts`` 2: query head h is zero outside half h % 2 of its entries (kernels may leave the other half out)."""
         T = q.shape[0]
         R, width = block_table.shape
         total_pages, _, page_size, _ = k_cache.shape
@@ -699,7 +761,8 @@ class NativeOps:
         self.launches += 1 if scratch is None else (decode_kernels if num_single == R else decode_kernels + 1)
         self.k.attention(_p(q), _p(k_cache), _p(v_cache), _p(block_table), width, _p(cu_q), _p(kv_len), _p(out), T, R,
                          nh, nkv, hd, page_size, total_pages, int(window), float(scale), _p(slopes), int(chunk), _p(sinks),
-                         float(softcap), int(max_q_len), int(max_kv_len), int(num_single), _p(scratch), _dt(q.dtype), self.fast,
+                         float(softcap), int(keep_first), int(parts), int(max_q_len), int(max_kv_len), int(num_single), _p(scratch),
+                         _dt(q.dtype), self.fast,
                          self._stream())
         return out
 
@@ -766,7 +829,7 @@ class NativeOps:
 
     def moe_combine(self, y, dest, wts, shared, gate, resid, ids=None, num_real=0, passthrough=None, shared_scale=1.0):
         """``resid[t] += sum_j wts[t, j] y[dest[t, j]] + shared_scale * gate[t] * shared[t]`` (no gate: 1).  With
-        ``ids``: a pair whose expert id is ``num_real`` or more reads ``passthrough[t]`` (32-bit ``[T, H]``) instead of
+        ``wts`` None: every weight 1.  ``ids``: a pair whose expert id is ``num_real`` or more reads ``passthrough[t]`` (32-bit ``[T, H]``) instead of
         a row of y (``y`` may be None when there are no other experts)."""
         T, H = resid.shape
         assert ids is None or (passthrough is not None and passthrough.shape == (T, H) and passthrough.is_contiguous()

@@ -6,7 +6,7 @@ import math
 import torch
 
 from ..registry import build_part, register_part
-from .base import CacheTensor, Mixer, PagedCache, PagedKV, ParamSpec, PartSpec, Runtime, StepContext
+from .base import CacheTensor, Mixer, PagedCache, PagedKV, ParamSpec, PartSpec, RequestState, Runtime, StepContext
 from .rope import rope_inv_freqs
 
 
@@ -275,7 +275,8 @@ class HeadNormedAttention(Mixer):
     heads), every key head likewise with ``k.norm``; then the rotation (``position``: any registered rotary encoding;
     its table, how many entries it turns and how it pairs them are the encoding's).  A score is ``(q . k) * scale``,
     and with ``softcap`` c then ``c tanh(score / c)``.
-    A query at p sees key ``j <= p`` iff ``p - j < window`` (when a window is given) and
+    A query at p sees key ``j <= p`` iff ``p - j < window`` (when a window is given; with ``keep_first`` the first
+    tokens of a request stay visible behind it) and
     ``floor(j / chunk) == floor(p / chunk)`` (when a chunk size is given; chunks are counted from position 0 of the
     request).  With ``sink`` the softmax's denominator also holds ``exp(sink_n)``, a learned logit per head that has
     no key and no value and is not scaled; ``sink_logit`` instead gives a logit that is a constant.  ``gate`` True or ``"head"``: head n's output is multiplied by
@@ -298,7 +299,7 @@ class HeadNormedAttention(Mixer):
                  qk_norm: bool | str = True, position: PartSpec | None = None, window: int | None = None,
                  chunk: int | None = None, sink: bool = False, gate: bool | str = False, out_scale: float = 1.0,
                  qkv_bias: bool = False, o_bias: bool = False, softcap: float | None = None,
-                 sink_logit: float | None = None, own_kv: bool = True):
+                 sink_logit: float | None = None, own_kv: bool = True, keep_first: int = 0):
         if heads % kv_heads:
             raise ValueError("heads must be a multiple of kv_heads")
         if gate not in (False, True, "head", "entry"):
@@ -317,6 +318,9 @@ class HeadNormedAttention(Mixer):
         self.softcap = float(softcap) if softcap else 0.0
         self.window = int(window) if window else None
         self.chunk = int(chunk) if chunk else None
+        self.keep = int(keep_first) if window else 0
+        if self.keep and self.chunk:
+            raise ValueError("kept first tokens go with a window, not with chunks")
         self.position = build_part("position", position) if position is not None else None
         need = max(self.d, self.dv)
         self.D = next((s for s in self._HEAD_SIZES if s >= need), -(-need // 8) * 8)
@@ -370,7 +374,7 @@ class HeadNormedAttention(Mixer):
         return min(spans) if spans else None
 
     def cache_need(self):
-        return PagedKV(self.G, self.D, self._span())
+        return PagedKV(self.G, self.D, self._span(), keep_first=self.keep)
 
     def forward(self, h, resid, ctx: StepContext, call: int):
         rt, ops, b = ctx.rt, ctx.rt.ops, ctx.batch
@@ -387,6 +391,8 @@ class HeadNormedAttention(Mixer):
                                      rt.dtype, amplitude=self.position.amplitude if rot is not None else 1.0,
                                      norm_after=self.norm_after)
         extra = {"softcap": self.softcap} if self.softcap else {}
+        if self.keep:
+            extra["keep_first"] = self.keep
         o = ops.attention(q, view.k, view.v, view.group.block_table, b.cu_q, b.kv_len, self.window or 0, self.scale,
                           H, G, self.D, b.max_q_len, b.max_kv_len, b.num_single, chunk=self.chunk or 0, sinks=self.sink,
                           **extra)
@@ -404,6 +410,90 @@ class HeadNormedAttention(Mixer):
             ops.add_vec_rows(resid, None, bias)
 
 
+class DifferentialAttention(Mixer):
+    """Grouped-query attention whose heads are the difference of two score maps over the same values.
+
+    ``q = W_q h`` holds ``heads`` x 2 maps x ``dim``, ``k = W_k h`` ``kv_heads`` x 2 maps x ``dim``, ``v = W_v h``
+    ``kv_heads`` x ``vdim`` (query head n reads key/value head ``n // (heads / kv_heads)``).  With ``conv_taps`` t every
+    channel of q, k and v first passes a causal convolution over time (``q.conv`` ``[channels, t]`` and so on; the last
+    tap meets the current token, zeros before the start), whose last t - 1 inputs are part of a request's state.  Every
+    map of q and k is divided by its root mean square and multiplied by ``q.norm`` / ``k.norm`` (``[dim]``, the same for
+    all heads and maps).  No positions enter the scores.  A score is ``(q . k) * scale``; a query at p sees ``j <= p``
+    with ``p - j < window`` (None: all) or ``j < keep_first``; a softmax per map.  With a1, a2 the two maps' outputs
+    and ``lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff`` (one number a layer), a head gives ``a1 - lambda a2`` divided
+    by its root mean square over ``vdim``, times ``1 - diff``.  With ``gate`` the heads side by side are multiplied entry
+    by entry by ``sigmoid(W_g h)``; then ``W_o``.
+
+    A stored key is the two maps' keys side by side, one in each half of D entries (D the larger of ``2 dim`` and
+    ``vdim``, rounded up to a size the tensor-core kernels take), and a map's query is zero in the other half: the
+    attention kernels then see ``2 heads`` query heads over ``kv_heads`` keys and values, and the values are stored and
+    read once for both maps."""
+
+    _HEAD_SIZES = (16, 32, 48, 64, 96, 128)
+    MAX_HEAD = 256
+
+    def __init__(self, hidden_size: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, eps: float,
+                 diff: float, conv_taps: int | None = None, window: int | None = None, keep_first: int = 0,
+                 gate: bool = True):
+        if heads % kv_heads:
+            raise ValueError("heads must be a multiple of kv_heads")
+        self.hidden, self.H, self.G, self.d, self.dv = int(hidden_size), int(heads), int(kv_heads), int(dim), int(vdim)
+        self.scale, self.eps, self.diff = float(scale), float(eps), float(diff)
+        self.taps = int(conv_taps) if conv_taps else 0
+        self.window = int(window) if window else None
+        self.keep = int(keep_first) if window else 0        # without a window nothing is ever out of sight
+        self.has_gate = bool(gate)
+        need = max(2 * self.d, self.dv)
+        self.D = next((s for s in self._HEAD_SIZES if s >= need), -(-need // 16) * 16)
+        if self.D > self.MAX_HEAD:
+            raise ValueError(f"two keys ({self.d} each) or a value ({self.dv}) do not fit in {self.MAX_HEAD} entries")
+        self.channels = 2 * (self.H + self.G) * self.d + self.G * self.dv       # of q, k and v
+        self.lam = 0.0
+        self.w_in = self.w_o = self.conv_w = self.qn = self.kn = None
+
+    def _rows(self):
+        return {"q": 2 * self.H * self.d, "k": 2 * self.G * self.d, "v": self.G * self.dv}
+
+    def param_specs(self):
+        specs = [ParamSpec(n, (r, self.hidden)) for n, r in self._rows().items()]
+        specs += [ParamSpec(n + ".norm", (self.d,), init="norm") for n in "qk"]
+        if self.taps:
+            specs += [ParamSpec(n + ".conv", (r, self.taps)) for n, r in self._rows().items()]
+        specs += [ParamSpec(n, (self.d,), init="bias") for n in ("lq1", "lk1", "lq2", "lk2")]
+        if self.has_gate:
+            specs.append(ParamSpec("g", (self.H * self.dv, self.hidden)))
+        return specs + [ParamSpec("o", (self.hidden, self.H * self.dv))]
+
+    def load(self, tensors, rt: Runtime):
+        self.w_in = torch.cat([rt.matrix(tensors[n]) for n in ["q", "k", "v"] + ["g"] * self.has_gate], dim=0).contiguous()
+        self.w_o = rt.matrix(tensors["o"])
+        self.qn, self.kn = rt.vector(tensors["q.norm"]), rt.vector(tensors["k.norm"])
+        if self.taps:           # [taps, channels]: neighbouring channels lie side by side
+            self.conv_w = torch.cat([rt.vector(tensors[n + ".conv"]) for n in "qkv"], dim=0).t().contiguous()
+        dot = lambda a, b: float((rt.vector(tensors[a]) * rt.vector(tensors[b])).sum())
+        self.lam = math.exp(dot("lq1", "lk1")) - math.exp(dot("lq2", "lk2")) + self.diff
+
+    def cache_need(self):
+        return PagedKV(self.G, self.D, self.window, keep_first=self.keep)
+
+    def state_need(self):
+        return {"conv": RequestState((self.taps - 1, self.channels))} if self.taps > 1 else None
+
+    def forward(self, h, resid, ctx: StepContext, call: int):
+        rt, ops, b = ctx.rt, ctx.rt.ops, ctx.batch
+        view = ctx.paged(call)
+        proj = ops.linear(h, self.w_in, None, torch.float32)               # [q | k | v | gate]
+        state = ctx.state(call, "conv") if self.taps > 1 else None
+        q = ops.map_norm_write(proj, self.conv_w, state, b, self.qn, self.kn, self.eps, view.group.slots, view.k, view.v,
+                               self.H, self.G, self.d, self.dv, self.D, rt.dtype)
+        o = ops.attention(q, view.k, view.v, view.group.block_table, b.cu_q, b.kv_len, self.window or 0, self.scale,
+                          2 * self.H, self.G, self.D, b.max_q_len, b.max_kv_len, b.num_single, keep_first=self.keep, parts=2)
+        gate = proj[:, self.channels:] if self.has_gate else None
+        ops.linear_add(ops.diff_norm_gate(o, gate, self.H, self.dv, self.D, self.lam, self.eps, 1.0 - self.diff), self.w_o,
+                       resid)
+
+
+register_part("mixer", "differential_attention", DifferentialAttention)
 register_part("mixer", "gqa_attention", GroupedQueryAttention)
 register_part("mixer", "head_normed_attention", HeadNormedAttention)
 register_part("mixer", "normed_biased_attention", NormedBiasedAttention)

@@ -50,11 +50,13 @@ class CacheTensor:
 class PagedCache:
     """What a mixer wants cached per token, in pages: any number of tensors (keys and values, or
     one latent vector, ...).  ``window`` None keeps every token, W keeps the last W (older pages go
-    back to the pool).  ``page_size`` None takes the engine's page size; layers whose window and
-    page size agree share a pool of pages and a block table."""
+    back to the pool) and, with ``keep_first`` k, the first k as well.  ``page_size`` None takes the
+    engine's page size; layers whose window, kept tokens and page size agree share a pool of pages and a
+    block table."""
     tensors: tuple[CacheTensor, ...]
     window: int | None = None
     page_size: int | None = None
+    keep_first: int = 0
 
     def elements_per_token(self) -> int:
         return sum(t.heads * t.width for t in self.tensors)
@@ -63,11 +65,12 @@ class PagedCache:
         return self.tensors == other.tensors and self.page_size == other.page_size
 
 
-def PagedKV(num_kv_heads: int, head_dim: int, window: int | None = None, page_size: int | None = None) -> PagedCache:
+def PagedKV(num_kv_heads: int, head_dim: int, window: int | None = None, page_size: int | None = None,
+            keep_first: int = 0) -> PagedCache:
     """The need of an attention mixer: per token ``num_kv_heads * head_dim`` keys (tensor ``k``)
     and as many values (tensor ``v``)."""
     return PagedCache((CacheTensor("k", int(num_kv_heads), int(head_dim)),
-                       CacheTensor("v", int(num_kv_heads), int(head_dim))), window, page_size)
+                       CacheTensor("v", int(num_kv_heads), int(head_dim))), window, page_size, int(keep_first))
 
 
 @dataclass(frozen=True)

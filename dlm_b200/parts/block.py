@@ -46,7 +46,8 @@ class PreNormBlock(Part):
 
 
 class ParallelBlock(PreNormBlock):
-    """``x += mixer(norm1(x)) + ffn(norm2(x))``: both sublayers read the same x, each through a norm of its own.
+    """``x += mixer(norm1(x)) + ffn(norm2(x))``: both sublayers read the same x, each through a norm of its own, or
+    (``norm2`` None with a feed-forward) both through ``norm1``, which then runs once.
     ``ffn`` None: the layer has no feed-forward (and no second norm).  The feed-forward runs first: its router may
     read the residual itself (through ``norm2``), which must still be the layer's input then; the mixer's input was
     normed before anything was added."""
@@ -56,15 +57,17 @@ class ParallelBlock(PreNormBlock):
         self.norm1 = build_part("norm", norm1)
         self.mixer = build_part("mixer", mixer)
         self.ffn = build_part("ffn", ffn) if ffn is not None else None
-        self.norm2 = build_part("norm", norm2) if ffn is not None else None
+        self.norm2 = build_part("norm", norm2) if ffn is not None and norm2 is not None else None
         self.names = {"norm1": "norm1.", "mixer": "mixer.", "norm2": "norm2.", "ffn": "ffn."}
         if names:
             self.names.update(names)
 
     def children(self):
         out = [(self.names["norm1"], self.norm1), (self.names["mixer"], self.mixer)]
+        if self.norm2 is not None:
+            out.append((self.names["norm2"], self.norm2))
         if self.ffn is not None:
-            out += [(self.names["norm2"], self.norm2), (self.names["ffn"], self.ffn)]
+            out.append((self.names["ffn"], self.ffn))
         return out
 
     def load(self, tensors, rt):
@@ -76,6 +79,11 @@ class ParallelBlock(PreNormBlock):
         rt = ctx.rt
         if self.ffn is None:
             self.mixer.forward(self.norm1.forward(resid, rt), resid, ctx, call)
+            return
+        if self.norm2 is None:
+            h = self.norm1.forward(resid, rt)
+            self.ffn.forward(h, resid, ctx, pre_norm=self.norm1)
+            self.mixer.forward(h, resid, ctx, call)
             return
         a, b = self.norm1.fusable_rms(), self.norm2.fusable_rms()
         both = self.norm1.pair_with(self.norm2)

@@ -71,6 +71,30 @@ class DenseActMLP(FeedForward):
         ops.linear_add(act, self.w_down, resid)
 
 
+class DenseClampedGLU(FeedForward):
+    """``resid += down · (g sigmoid(alpha g) (u + shift))`` with ``g = min(gate·h, limit)`` and ``u`` the up product
+    clamped to ``[-limit, limit]``, no biases; the gate is the first product's epilogue."""
+
+    def __init__(self, hidden_size: int, intermediate_size: int, limit: float, alpha: float = 1.702, shift: float = 1.0,
+                 names: dict[str, str] | None = None):
+        self.hidden, self.inter = int(hidden_size), int(intermediate_size)
+        self.limit, self.alpha, self.shift = float(limit), float(alpha), float(shift)
+        self.names = {"gate": "gate", "up": "up", "down": "down"}
+        if names:
+            self.names.update(names)
+        self.w_gate_up = self.w_down = self.constants = None
+
+    param_specs = DenseSwiGLU.param_specs
+
+    def load(self, tensors, rt: Runtime):
+        DenseSwiGLU.load(self, tensors, rt)
+        self.constants = rt.vector(torch.tensor([self.limit, self.alpha, self.shift], dtype=torch.float32))
+
+    def forward(self, h, resid, ctx: StepContext, pre_norm=None):
+        ops = ctx.rt.ops
+        ops.linear_add(ops.linear_clamped_glu(h, self.w_gate_up, self.constants), self.w_down, resid)
+
+
 class SoftmaxTopKMoE(FeedForward):
     """Routed experts as the reference computes them (src/forward/cpu.rs:980-1048): router
     logits in 32-bit from the 32-bit normalised residual, softmax over all experts, the k largest probabilities (ties: lower
@@ -80,12 +104,16 @@ class SoftmaxTopKMoE(FeedForward):
     tensor is required; False, there is none and the factor is 1; None, the checkpoint decides:
     a missing gate tensor means the factor 1 (src/forward/cpu.rs:1032-1041).
 
+    ``score`` "sigmoid": the scores are the logistic function of each logit instead of a softmax over the experts.
+    ``weigh`` "input": a chosen expert sees the token's row times its weight, and its output is added as it is.
+
     At load the experts are stacked into ``[E, 2I, H]`` (gate and up rows interleaved) and
     ``[E, H, I]``; the router and the shared gate become one ``[E (+1), H]`` matrix."""
 
     def __init__(self, hidden_size: int, num_experts: int, top_k: int, expert_intermediate_size: int,
                  norm_topk_prob: bool, shared_intermediate_size: int | None = None,
-                 shared_gate: bool | None = True, router_bias: bool = False, names: dict[str, str] | None = None):
+                 shared_gate: bool | None = True, router_bias: bool = False, names: dict[str, str] | None = None,
+                 score: str = "softmax", weigh: str = "output"):
         """``router_bias``: the router has a bias (tensor ``names["router_bias"]``) that is added to its logits; with
         ``norm_topk_prob`` the weights are then the softmax over the chosen logits.  ``names``: the tensors' names
         (``{e}`` stands for the expert's number), by default the ones of Qwen2-MoE checkpoints."""
@@ -96,6 +124,11 @@ class SoftmaxTopKMoE(FeedForward):
                       "shared_gate": "shared_expert_gate.weight"}
         if names:
             self.names.update(names)
+        if score not in ("softmax", "sigmoid") or weigh not in ("output", "input"):
+            raise ValueError(f"unknown score {score!r} or place of the weight {weigh!r}")
+        if router_bias and score != "softmax":
+            raise ValueError("a router bias goes with softmax scores")
+        self.score, self.weigh_input = score, weigh == "input"
         self.router_bias = bool(router_bias)
         self.b_router = None
         self.hidden, self.E, self.k, self.I = int(hidden_size), int(num_experts), int(top_k), int(expert_intermediate_size)
@@ -148,7 +181,9 @@ class SoftmaxTopKMoE(FeedForward):
         ops = ctx.rt.ops
         rms = pre_norm.fusable_rms() if pre_norm is not None else None
         shared = None
-        bias = {"logit_bias": self.b_router} if self.b_router is not None else {}
+        extra = {"logit_bias": self.b_router} if self.b_router is not None else {}
+        if self.score != "softmax":
+            extra["score"] = self.score
         branch = ops.branch(h.shape[0])
         if self.Is:
             # the shared expert needs nothing from the router: it may run beside the routed experts
@@ -162,11 +197,13 @@ class SoftmaxTopKMoE(FeedForward):
             # one, the norm's or the shared expert's, only reads it)
             ids, wts, gate, offsets, rows, dest = ops.route(resid, self.w_router, self.E, self.k, self.norm,
                                                             self.has_gate, norm_weight=rms[0], eps=rms[1],
-                                                            input_settled=True, **bias)
+                                                            input_settled=True, **extra)
         else:
             x = h if pre_norm is None else pre_norm.forward(resid, ctx.rt, out_dtype=torch.float32)
             ids, wts, gate, offsets, rows, dest = ops.route(x, self.w_router, self.E, self.k, self.norm, self.has_gate,
-                                                            **bias)
+                                                            **extra)
+        if self.weigh_input:
+            h, rows, wts = ops.weigh_rows(h, wts, dest), None, None
         act = ops.grouped_swiglu(h, self.w_gate_up, offsets, rows)
         y = ops.grouped_linear(act, self.w_down, offsets)
         branch.join()
@@ -294,4 +331,6 @@ register_part("ffn", "table_experts", TableRoutedExperts)
 register_part("ffn", "routed_act_experts", RoutedActExperts)
 register_part("ffn", "swiglu_dense", DenseSwiGLU)
 register_part("ffn", "dense_act", DenseActMLP)
+register_part("ffn", "clamped_glu_dense", DenseClampedGLU)
 register_part("ffn", "moe_softmax_topk", SoftmaxTopKMoE)
+register_part("ffn", "moe_topk", SoftmaxTopKMoE)

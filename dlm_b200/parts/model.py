@@ -37,6 +37,8 @@ class ModelSpec:
     order: list[LayerCall] | None = None # None: every layer once, in index order
     embed_position: PartSpec | None = None   # a position encoding that acts on the embedded tokens
     embed_position_prefix: str = ""          # tensor-name prefix of that encoding's own tensors (if it has any)
+    embed_norm: PartSpec | None = None       # a norm on the embedded tokens (positions added): what the first layer gets
+    embed_norm_prefix: str = ""              # tensor-name prefix of that norm's tensors
     embed_scale: float = 1.0                 # the embedded tokens are multiplied by this
     residual_streams: int | None = None      # S: blocks get ``[T, S, hidden]`` (S equal copies at the start, summed at the end)
     pass_entry: PartSpec | None = None       # what makes the input of a repeated run's pass (calls with ``enters_pass``)
@@ -72,6 +74,7 @@ class DecoderModel:
         self.blocks = [build_part("block", bs) for bs in spec.layers]
         self.final_norm = build_part("norm", spec.final_norm)
         self.embed_position = build_part("position", spec.embed_position) if spec.embed_position else None
+        self.embed_norm = build_part("norm", spec.embed_norm) if spec.embed_norm else None
         self.pass_entry = build_part("entry", spec.pass_entry) if spec.pass_entry else None
         self.order = list(spec.order) if spec.order is not None else [LayerCall(i) for i in range(len(self.blocks))]
         for ci, c in enumerate(self.order):
@@ -99,6 +102,9 @@ class DecoderModel:
         if self.embed_position is not None:
             for p in self.embed_position.param_specs():
                 out[s.embed_position_prefix + p.name] = replace(p, name=s.embed_position_prefix + p.name)
+        if self.embed_norm is not None:
+            for p in self.embed_norm.param_specs():
+                out[s.embed_norm_prefix + p.name] = replace(p, name=s.embed_norm_prefix + p.name)
         if self.pass_entry is not None:
             for p in self.pass_entry.param_specs():
                 out[s.pass_entry_prefix + p.name] = replace(p, name=s.pass_entry_prefix + p.name)
@@ -141,6 +147,9 @@ class DecoderModel:
         if self.embed_position is not None:
             mine = {s.embed_position_prefix + p.name for p in self.embed_position.param_specs()}
             self.embed_position.load({n[len(s.embed_position_prefix):]: get(n) for n in names if n in mine}, rt)
+        if self.embed_norm is not None:
+            mine = {s.embed_norm_prefix + p.name for p in self.embed_norm.param_specs()}
+            self.embed_norm.load({n[len(s.embed_norm_prefix):]: get(n) for n in names if n in mine}, rt)
         if self.pass_entry is not None:
             mine = {s.pass_entry_prefix + p.name for p in self.pass_entry.param_specs()}
             self.pass_entry.load({n[len(s.pass_entry_prefix):]: get(n) for n in names if n in mine}, rt)
@@ -162,8 +171,9 @@ class DecoderModel:
             out.append((block.mixer.cache_need(), state, owner))
         for ci, (need, _, owner) in enumerate(out):
             own = out[owner][0]
-            if owner != ci and own.window is not None and (need.window is None or need.window > own.window):
-                out[owner] = (replace(own, window=need.window), *out[owner][1:])
+            if owner != ci and own.window is not None:
+                window = None if need.window is None else max(need.window, own.window)
+                out[owner] = (replace(own, window=window, keep_first=max(need.keep_first, own.keep_first)), *out[owner][1:])
         return out
 
     # ---------------------------------------------------------------- step
@@ -187,6 +197,8 @@ class DecoderModel:
         x = ops.embed(batch.tokens, self.embed, s.embed_scale) if s.embed_scale != 1.0 else ops.embed(batch.tokens, self.embed)
         if self.embed_position is not None:
             self.embed_position.on_embed(x, batch.positions, rt)
+        if self.embed_norm is not None:
+            x = self.embed_norm.forward(x, rt, out_dtype=torch.float32)
         if s.residual_streams is not None:
             x = ops.streams_expand(x, s.residual_streams)
         # a model with repeated passes keeps the embedded tokens: blocks change x in place

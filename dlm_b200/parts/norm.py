@@ -11,18 +11,23 @@ class RMSNorm(Norm):
     """``out = (x / sqrt(mean(x^2) + eps)) * weight`` with 32-bit statistics
     (src/forward/cpu.rs:934-942); the result is stored in the activation dtype."""
 
-    def __init__(self, size: int, eps: float, param: str = "weight", scale: float = 1.0):
+    def __init__(self, size: int, eps: float, param: str = "weight", scale: float = 1.0, offset: float = 0.0):
         """``param``: the weight tensor's name relative to the part's prefix ("" when the prefix is the
         whole name).  ``scale``: a factor on the output (it joins the 32-bit weight at load): a model whose logits
-        are its head's product times a constant gives that constant to its final norm."""
+        are its head's product times a constant gives that constant to its final norm.  ``offset``: what is added to
+        the stored weight, in 32-bit at load (1 for checkpoints that store a weight's distance from one)."""
         self.size, self.eps, self.param, self.scale = int(size), float(eps), str(param), float(scale)
+        self.offset = float(offset)
         self.weight: torch.Tensor | None = None
 
     def param_specs(self):
-        return [ParamSpec(self.param, (self.size,), init="norm")]
+        # (an offset of 1 moves the stored weight to around zero: drawn as a bias is)
+        return [ParamSpec(self.param, (self.size,), init="bias" if self.offset else "norm")]
 
     def load(self, tensors, rt: Runtime):
         self.weight = rt.vector(tensors[self.param])
+        if self.offset != 0.0:
+            self.weight = (self.weight + self.offset).contiguous()
         if self.scale != 1.0:
             self.weight = (self.weight * self.scale).contiguous()
 

@@ -87,4 +87,4 @@ def _ensure_builtin() -> None:
         return
     _builtin_done = True
     from . import parts  # noqa: F401  registers the built-in parts
-    from .models import faguzen, qwen2_moe, salolorn, zasazen, zepilorn, zesapel  # noqa: F401  register the architectures
+    from .models import faguzen, gakenex, qwen2_moe, salolorn, zasazen, zepilorn, zesapel  # noqa: F401  register the architectures

@@ -324,6 +324,52 @@ class PlainOps:
             v_cache[page, :, off, :] = pad(v, (0, D - dv))[ok].to(v_cache.dtype)
         return pad(q, (0, D - d)).reshape(T, nh * D).to(out_dtype)
 
+    def map_norm_write(self, proj, conv_w, state, batch, qn_w, kn_w, eps, slots, k_cache, v_cache, H, G, d, dv, D, out_dtype):
+        T = proj.shape[0]
+        C = 2 * (H + G) * d + G * dv
+        x = proj[:, :C]
+        if conv_w is not None:
+            if state is None:
+                state = torch.zeros((int(batch.state_slot.max()) + 1, 0, C))
+            x = self.causal_conv(x, conv_w.t(), None, state, batch, False, False, torch.float32)
+        rms = lambda v, w: (v * (1.0 / torch.sqrt((v * v).mean(-1, keepdim=True) + eps))) * w
+        q = rms(x[:, :2 * H * d].reshape(T, H, 2, d), qn_w)
+        k = rms(x[:, 2 * H * d:2 * (H + G) * d].reshape(T, G, 2, d), kn_w)
+        v = x[:, 2 * (H + G) * d:].reshape(T, G, dv)
+        half = D // 2
+        qo = torch.zeros(T, H, 2, D)
+        ko, vo = torch.zeros(T, G, D), torch.zeros(T, G, D)
+        for m in range(2):
+            qo[:, :, m, m * half:m * half + d] = q[:, :, m]
+            ko[:, :, m * half:m * half + d] = k[:, :, m]
+        vo[..., :dv] = v
+        ps = k_cache.shape[2]
+        sl = slots.long()
+        ok = sl >= 0
+        k_cache[sl[ok] // ps, :, sl[ok] % ps, :] = ko[ok].to(k_cache.dtype)
+        v_cache[sl[ok] // ps, :, sl[ok] % ps, :] = vo[ok].to(v_cache.dtype)
+        return qo.reshape(T, 2 * H * D).to(out_dtype)
+
+    def diff_norm_gate(self, o, gate, H, dv, D, lam, eps, factor):
+        T = o.shape[0]
+        a = _f(o).reshape(T, H, 2, D)[..., :dv]
+        c = a[:, :, 0] - lam * a[:, :, 1]
+        c = (c * (factor / torch.sqrt((c * c).mean(-1, keepdim=True) + eps))).reshape(T, H * dv)
+        return (c if gate is None else c * torch.sigmoid(gate)).to(o.dtype)
+
+    def weigh_rows(self, h, wts, dest):
+        T, k = dest.shape
+        out = torch.zeros((T * k, h.shape[1]), dtype=h.dtype, device=h.device)
+        for j in range(k):
+            out[dest[:, j].long()] = (_f(h) * wts[:, j:j + 1]).to(h.dtype)
+        return out
+
+    def linear_clamped_glu(self, a, w_gate_up, constants):
+        limit, alpha, shift = (float(c) for c in constants)
+        acc = _f(a) @ _f(w_gate_up).T
+        g, u = acc[:, 0::2].clamp(max=limit), acc[:, 1::2].clamp(-limit, limit)
+        return (g * torch.sigmoid(alpha * g) * (u + shift)).to(a.dtype)
+
     def head_gate(self, o, gate, nh, D, factor=1.0):
         T = o.shape[0]
         g = factor * torch.sigmoid(gate)
@@ -414,6 +460,8 @@ class PlainOps:
 
     def grouped_swiglu(self, a, w_gate_up, offsets, rows):
         E, N, K = w_gate_up.shape
+        if rows is None:                        # already grouped
+            rows = torch.arange(a.shape[0], device=a.device)
         out = torch.zeros((rows.numel(), N // 2), dtype=a.dtype, device=a.device)
         off = offsets.tolist()
         for e in range(E):
@@ -478,7 +526,7 @@ class PlainOps:
         return q.reshape(T, Q).to(out_dtype)
 
     def attention(self, q, k_cache, v_cache, block_table, cu_q, kv_len, window, scale, nh, nkv, hd, max_q_len,
-                  max_kv_len, num_single=0, slopes=None, chunk=0, sinks=None, softcap=0.0):
+                  max_kv_len, num_single=0, slopes=None, chunk=0, sinks=None, softcap=0.0, keep_first=0, parts=1):
         T = q.shape[0]
         ps = k_cache.shape[2]
         out = torch.zeros((T, nh * hd), dtype=torch.float32, device=q.device)
@@ -492,7 +540,8 @@ class PlainOps:
             lo = max(0, first - window + 1) if window > 0 else 0
             if chunk > 0:
                 lo = max(lo, (first // chunk) * chunk)
-            pos = torch.arange(lo, n, device=q.device)
+            kept = min(keep_first, lo) if window > 0 else 0
+            pos = torch.cat([torch.arange(kept, device=q.device), torch.arange(lo, n, device=q.device)])
             pages = block_table[r, (pos // ps).long()].long()
             assert int(pages.min()) >= 0, "a visible key has no page"
             k = _f(k_cache[pages, :, pos % ps, :])          # [n - lo, nkv, hd]
@@ -501,7 +550,7 @@ class PlainOps:
             qpos = torch.arange(first, n, device=q.device)
             ok = pos[None, :] <= qpos[:, None]
             if window > 0:
-                ok &= (qpos[:, None] - pos[None, :]) < window
+                ok &= ((qpos[:, None] - pos[None, :]) < window) | (pos[None, :] < keep_first)
             if chunk > 0:
                 ok &= torch.div(pos, chunk, rounding_mode="floor")[None, :] == torch.div(qpos, chunk, rounding_mode="floor")[:, None]
             for h in range(nh):
@@ -611,7 +660,7 @@ class PlainOps:
                 src = passthrough.clone()
                 if y is not None and bool(real.any()):
                     src[real] = y[dest[real, j].long()]
-            acc = acc + wts[:, j:j + 1] * src
+            acc = acc + (src if wts is None else wts[:, j:j + 1] * src)
         if shared is not None:
             g = gate[:, None] if gate is not None else 1.0
             acc = acc + (g * shared_scale) * shared
