@@ -134,7 +134,7 @@ class PlainGakenex:
         return h, a, weighted_input_experts(h, p, mlp["router"]["top"], r)
 
     def router_margins(self, tokens):
-        """Per position the smallest gap, over all layers with a router, between the last chosen score and the next."""
+        """Per position the smallest gap, over all layers with a router, between the last chosen logit and the next."""
         x = self.embedded(tokens)
         gap = torch.full((len(tokens),), float("inf"), dtype=self.dtype)
         for i, spec in enumerate(self.cfg["layers"]):
@@ -142,8 +142,8 @@ class PlainGakenex:
             mlp = spec.get("mlp")
             if mlp and mlp["kind"] == "moe" and mlp["router"]["top"] < mlp["router"]["experts"]:
                 top = mlp["router"]["top"]
-                s = torch.sort(sigmoid(h @ self.t[f"l{i}.mlp.router"].T), dim=-1, descending=True).values
-                gap = torch.minimum(gap, s[:, top - 1] - s[:, top])
+                z = torch.sort(h @ self.t[f"l{i}.mlp.router"].T, dim=-1, descending=True).values
+                gap = torch.minimum(gap, z[:, top - 1] - z[:, top])
             x = x + (a + f)
         return gap
 
