@@ -14,6 +14,7 @@ continuous-batching workload on the windowed variant of the model (`serving`).
     python bench.py --workload salolorn     # the Salolorn design beside a dense Qwen2 at equal sizes, and its kernels alone
     python bench.py --workload faguzen      # the Faguzen design beside Qwen2-MoE at equal sizes, and its kernels alone
     python bench.py --workload zepilorn     # the Zepilorn design beside a dense Qwen2 at equal sizes, and its kernels alone
+    python bench.py --workload gakenex      # the Gakenex design beside Qwen2-MoE at equal sizes, and its kernels alone
 
 A step is one decode step of the whole batch.  One JSON line is printed.
 """
@@ -1514,6 +1515,200 @@ def run_zepilorn(args, pk) -> dict:
     return out
 
 
+def gakenex_config(width, vocab=32768, window=512, keep=64):
+    """Four layers of the design at a real model's layer sizes: two score maps of 64 over values of 128 a head, four query
+    heads a key/value head, four taps on queries, keys and values, a window that keeps the first tokens; a clamped gated
+    feed-forward three times the width and 16 experts of half the width (two a token), in turn."""
+    heads = width // 128
+    mixer = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 64, "vdim": 128, "scale": 64 ** -0.5, "diff": 0.35,
+             "conv": 4, "mask": {"size": window, "keep_first": keep}}
+    mlps = ({"kind": "dense", "ff": 3 * width, "limit": 7.0},
+            {"kind": "moe", "router": {"experts": 16, "top": 2}, "expert": {"ff": width // 2}})
+    return {"architecture": "Gakenex", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "max_positions": 8192,
+            "logit_softcap": 30.0, "layers": [{"type": "attention", "mixer": mixer, "mlp": mlps[i % 2]} for i in range(4)]}
+
+
+def qwen_config_like_gakenex(z):
+    """Qwen2-MoE with the same width, vocabulary and layers, the same dense and routed feed-forwards in turn (no shared
+    expert), and attention heads of the same number and value size over the same window."""
+    att, ff, moe = z["layers"][0]["mixer"], z["layers"][0]["mlp"], z["layers"][1]["mlp"]
+    n = len(z["layers"])
+    return dict(architectures=["Qwen2MoeForCausalLM"], model_type="qwen2_moe", num_hidden_layers=n,
+                hidden_size=z["width"], num_attention_heads=att["heads"], num_key_value_heads=att["kv_heads"],
+                head_dim=att["vdim"], num_experts=moe["router"]["experts"], num_experts_per_tok=moe["router"]["top"],
+                moe_intermediate_size=moe["expert"]["ff"], shared_expert_intermediate_size=0, norm_topk_prob=False,
+                decoder_sparse_step=1, mlp_only_layers=[i for i in range(n) if i % 2 == 0], intermediate_size=ff["ff"],
+                vocab_size=z["vocab"], rope_theta=1e6, rms_norm_eps=1e-6, use_sliding_window=True,
+                sliding_window=att["mask"]["size"], max_window_layers=0, tie_word_embeddings=True,
+                max_position_embeddings=8192)
+
+
+def gakenex_kernels(z, pk, batch, context, prefill_tokens):
+    """Each kernel of the design alone at the layer sizes of `z`, beside the like kernel of an existing model at the
+    same sizes: a prompt of `prefill_tokens` tokens of one request, and a decode step of `batch` requests at `context`
+    tokens.  Microseconds (median of 5, the cache flushed before each), the bytes the kernel has to move at least,
+    and that over time over the measured copy bandwidth; attentions and products also with their flops."""
+    from types import SimpleNamespace
+
+    import torch
+
+    from dlm_b200.ops import native_ops
+    ops = native_ops(fast=True)
+    dev, bf = "cuda", torch.bfloat16
+    W, V = z["width"], z["vocab"]
+    att, ff, moe = z["layers"][0]["mixer"], z["layers"][0]["mlp"]["ff"], z["layers"][1]["mlp"]
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    i32 = dict(dtype=torch.int32, device=dev)
+    rows = {}
+
+    def timed(name, case, fn, nbytes, flop=None):
+        ts = []
+        for _ in range(6):
+            _flush(torch, flush)
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record()
+            fn()
+            e1.record()
+            torch.cuda.synchronize()
+            ts.append(e0.elapsed_time(e1))
+        us = statistics.median(ts[1:]) * 1e3
+        row = {"us": round(us, 1), "mbytes": round(nbytes / 1e6, 2),
+               "frac_of_copy": round(nbytes / (us * 1e-6) / 1e9 / pk["hbm_gbs"], 3)}
+        if flop is not None:
+            row["gflop"] = round(flop / 1e9, 2)
+            row["frac_of_bf16_peak"] = round(flop / (us * 1e-6) / (pk["bf16_tflops"] * 1e12), 4)
+        rows.setdefault(name, {})[case] = row
+
+    with ops.dependent_launch(False):
+        for case, lens, start in (("prefill", [prefill_tokens], 0), ("decode", [1] * batch, context)):
+            T, R = sum(lens), len(lens)
+            cu = [0]
+            for n in lens:
+                cu.append(cu[-1] + n)
+            single = sum(1 for n in lens if n == 1)
+            b = SimpleNamespace(num_requests=R, num_single=single, cu_q=torch.tensor(cu, **i32),
+                                state_slot=torch.arange(R, **i32),
+                                token_req=torch.tensor([r for r, n in enumerate(lens) for _ in range(n)], **i32),
+                                positions=torch.tensor([start + i for n in lens for i in range(n)], **i32))
+            held = start + max(lens)
+            pages_each = -(-held // 64)
+            table = torch.arange(R * pages_each, **i32).reshape(R, pages_each)
+            slots = torch.cat([table[r, (start + torch.arange(n, device=dev)) // 64] * 64
+                               + (start + torch.arange(n, device=dev)) % 64 for r, n in enumerate(lens)]).to(torch.int32)
+            kv_len = torch.tensor([start + n for n in lens], **i32)
+            # ---- from token ids to the first layer's input
+            ids = torch.randint(0, V, (T,), **i32)
+            emb, pos = (torch.randn(V, W, device=dev).to(bf), torch.randn(8192, W, device=dev).to(bf))
+            nw = torch.randn(W, device=dev)
+
+            def entry():
+                x = ops.embed(ids, emb)
+                ops.add_rows(x, pos, b.positions)
+                return ops.rmsnorm(x, nw, 1e-6, torch.float32)
+            timed("embedding, positions and norm", case, entry, T * W * 8)
+            timed("embedding (Qwen2's)", case, lambda: ops.embed(ids, emb), T * W * 6)
+            # ---- the two-map head: convolution, norms and write; attention; difference, norm and gate
+            H, G, d, dv, taps = att["heads"], att["kv_heads"], att["dim"], att["vdim"], att["conv"]
+            D = max(2 * d, dv)
+            window, keep = att["mask"]["size"], att["mask"]["keep_first"]
+            C = 2 * (H + G) * d + G * dv
+            k_cache = (torch.randn(R * pages_each + 1, G, 64, D, device=dev) * 0.3).to(bf)
+            v_cache = (torch.randn(R * pages_each + 1, G, 64, D, device=dev) * 0.3).to(bf)
+            proj = torch.randn(T, C + H * dv, device=dev)
+            conv_w, qn = torch.randn(taps, C, device=dev), torch.randn(d, device=dev)
+            state = torch.zeros(R + 1, taps - 1, C, device=dev)
+            io = T * C * 4 + T * (2 * H + 2 * G) * D * 2 + 2 * R * (taps - 1) * C * 4
+            write = lambda: ops.map_norm_write(proj, conv_w, state, b, qn, qn, 1e-6, slots, k_cache, v_cache, H, G, d, dv, D, bf)
+            timed("map_norm_write (convolution, norm per map, write)", case, write, io)
+            hp = torch.randn(T, (H + 2 * G) * D, device=dev)
+            dn, freq = torch.randn(D, device=dev), torch.tensor([1e6 ** (-2.0 * i / D) for i in range(D // 2)], device=dev)
+            timed("head_norm_rope_write (Salolorn's norm per head, rotation, write)", case,
+                  lambda: ops.head_norm_rope_write(hp, b.positions, dn, dn, 1e-6, freq, D, False, slots, k_cache, v_cache, H, G,
+                                                   D, D, D, bf), T * (H + 2 * G) * D * 6)
+            full = torch.zeros(R + 1, taps - 1, C, device=dev)
+            conv_wt = conv_w.t().contiguous()
+            timed("causal_conv alone (Zesapel's)", case,
+                  lambda: ops.causal_conv(proj[:, :C], conv_wt, None, full, b, False, False, torch.float32),
+                  T * C * 8 + 2 * R * (taps - 1) * C * 4)
+            q = write()
+            see = lambda p: min(window, p + 1) + min(keep, max(0, p + 1 - window))
+            keys = sum(see(start + i) for n in lens for i in range(n))
+            span = see(held - 1) if case == "decode" else held
+            nbytes = R * span * G * D * 4 + T * 2 * H * D * 4
+            timed("attention, two maps, window with kept tokens", case,
+                  lambda: ops.attention(q, k_cache, v_cache, table, b.cu_q, kv_len, window, att["scale"], 2 * H, G, D, max(lens),
+                                        held, single, keep_first=keep, parts=2), nbytes, flop=2.0 * keys * 2 * H * (d + dv))
+            timed("the same, the kernel not told that a query fills half a head", case,
+                  lambda: ops.attention(q, k_cache, v_cache, table, b.cu_q, kv_len, window, att["scale"], 2 * H, G, D, max(lens),
+                                        held, single, keep_first=keep), nbytes, flop=2.0 * keys * 2 * H * (d + dv))
+            wkeys = sum(min(window, start + i + 1) for n in lens for i in range(n))
+            qh = torch.randn(T, 2 * H * D, device=dev).to(bf)
+            timed("attention over a window, as many heads of 128 (Qwen2's)", case,
+                  lambda: ops.attention(qh, k_cache, v_cache, table, b.cu_q, kv_len, window, att["scale"], 2 * H, G, D, max(lens),
+                                        held, single), R * (min(window, held) if case == "decode" else held) * G * D * 4
+                  + T * 2 * H * D * 4, flop=2.0 * wkeys * 2 * H * 2 * D)
+            o = torch.randn(T, 2 * H * D, device=dev).to(bf)
+            gate = proj[:, C:]
+            timed("diff_norm_gate (difference of the maps, norm, gate)", case,
+                  lambda: ops.diff_norm_gate(o, gate, H, dv, D, 0.5, 1e-6, 0.65), T * H * (2 * dv * 2 + dv * 4 + dv * 2))
+            o1, g1 = torch.randn(T, H * dv, device=dev).to(bf), torch.randn(T, H * dv, device=dev)
+            timed("entry_gate (Faguzen's)", case, lambda: ops.entry_gate(o1, g1, H, dv, dv), T * H * dv * 8)
+            o32, n1 = torch.randn(T, H * dv, device=dev), torch.randn(H * dv, device=dev)
+            timed("gated_rmsnorm per head, sigmoid gate (Zesapel's)", case,
+                  lambda: ops.gated_rmsnorm(o32, g1, n1, H, 1e-6, "sigmoid_after", bf), T * H * dv * 10)
+            # ---- feed-forwards
+            h = torch.randn(T, W, device=dev).to(bf)
+            wgu = (torch.randn(2 * ff, W, device=dev) * 0.02).to(bf)
+            const = torch.tensor([7.0, 1.702, 1.0], device=dev)
+            nb, fl = (2 * ff * W + T * (W + ff)) * 2, 4.0 * T * W * ff
+            timed("gate and up product, clamped gate", case, lambda: ops.linear_clamped_glu(h, wgu, const), nb, flop=fl)
+            timed("gate and up product, silu (Qwen2's)", case, lambda: ops.linear_swiglu(h, wgu), nb, flop=fl)
+            E, k, I = moe["router"]["experts"], moe["router"]["top"], moe["expert"]["ff"]
+            wr = (torch.randn(E, W, device=dev) * 0.02).to(bf)
+            we, wd = (torch.randn(E, 2 * I, W, device=dev) * 0.02).to(bf), (torch.randn(E, W, I, device=dev) * 0.02).to(bf)
+            resid = torch.randn(T, W, device=dev)
+            used = min(E, T * k)
+            for name, score in (("router, sigmoid scores", "sigmoid"), ("router, softmax scores (Qwen2's)", "softmax")):
+                timed(name, case, lambda: ops.route(resid, wr, E, k, 0, False, norm_weight=nw, eps=1e-6, score=score),
+                      T * W * 4 + E * W * 2)
+            _, wts, _, offs, rws, dest = ops.route(resid, wr, E, k, 0, False, norm_weight=nw, eps=1e-6, score="sigmoid")
+            timed("weigh_rows", case, lambda: ops.weigh_rows(h, wts, dest), T * W * 2 + T * k * W * 2)
+            gathered = torch.empty(T * k, W, dtype=bf, device=dev)
+            timed("gather_rows (Qwen2's on prompts)", case,
+                  lambda: ops.k.gather_rows(h.data_ptr(), rws.data_ptr(), gathered.data_ptr(), T * k, W, 1, ops._stream()),
+                  T * W * 2 + T * k * W * 2)
+            nb, fl = (used * 2 * I * W + T * k * (W + I)) * 2, 4.0 * T * k * W * I
+            timed("experts' gate and up product, rows weighted before", case,
+                  lambda: ops.grouped_swiglu(ops.weigh_rows(h, wts, dest), we, offs, None), nb, flop=fl)
+            timed("experts' gate and up product (Qwen2's)", case, lambda: ops.grouped_swiglu(h, we, offs, rws), nb, flop=fl)
+            act = ops.grouped_swiglu(h, we, offs, rws)
+            y = ops.grouped_linear(act, wd, offs)
+            timed("moe_combine, no weights", case, lambda: ops.moe_combine(y, dest, None, None, None, resid), T * W * (k * 4 + 8))
+            timed("moe_combine (Qwen2's)", case, lambda: ops.moe_combine(y, dest, wts, None, None, resid), T * W * (k * 4 + 8))
+    ops.check_errors()
+    return rows
+
+
+def run_gakenex(args, pk) -> dict:
+    sampler = ClockSampler()
+    sampler.start()
+    t0 = time.time()
+    out = {"workload": "gakenex", "dtype": "bf16", "data": "synthetic: seeded uniform token ids, random weights N(0, 0.02)",
+           "peaks": pk, "sizes": {}, "l2": "a buffer larger than L2 is written before every timed step"}
+    for width in (1024, 2048, 4096):
+        z = gakenex_config(width)
+        q = qwen_config_like_gakenex(z)
+        out["sizes"][str(width)] = {
+            "layers": len(z["layers"]), "gakenex": measure_engine(z, args.batch, args.prompt_len, args.steps, 2048),
+            "qwen2_moe": measure_engine(q, args.batch, args.prompt_len, args.steps, 2048)}
+    out["kernels_width_2048"] = gakenex_kernels(gakenex_config(2048), pk, args.batch, args.prompt_len, 2048)
+    t1 = time.time()
+    time.sleep(0.2)
+    sampler.stop()
+    out["clocks"] = sampler.summary(t0, t1)
+    return out
+
+
 def layers_that_fit(raw, want, reserve_gb=40.0):
     """As many layers of `raw` (at most `want`) as the free device memory holds beside `reserve_gb` for
     the cache pool, the head, graphs and activations."""
@@ -1574,7 +1769,7 @@ def main() -> int:
     ap.add_argument("--no-extras", action="store_true", help="skip `sizes_57b` and `serving`")
     ap.add_argument("--only-prefill", action="store_true", help="measure the 2,048-token prefill alone (for profiles)")
     ap.add_argument("--workload", default="decode", choices=["decode", "serving", "sweep", "kernels", "zesapel", "zasazen", "salolorn", "faguzen",
-                                                              "zepilorn"],
+                                                              "zepilorn", "gakenex"],
                     help="serving: the continuous-batching workload on the windowed model, instead of the default line; "
                          "sweep: decode at contexts of 1k to 32k and prefill of longer prompts, a line of its own; "
                          "kernels: the weight-streaming product alone")
@@ -1619,6 +1814,9 @@ def main() -> int:
         return 0
     if args.workload == "zepilorn":
         print(json.dumps(run_zepilorn(args, pk)))
+        return 0
+    if args.workload == "gakenex":
+        print(json.dumps(run_gakenex(args, pk)))
         return 0
     max_batch = 64 if not args.no_points else args.batch
     m = Measurement(MODEL, args.layers, args.prompt_len, args.context, max_batch, pk, page=args.page_size)

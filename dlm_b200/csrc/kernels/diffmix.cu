@@ -283,6 +283,7 @@ void diff_norm_gate_of(const void* o, const float* gate, int ldg, void* out, lon
 }
 
 bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
+bool aligned8(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 7) == 0; }
 
 }  // namespace
 
@@ -301,9 +302,9 @@ void map_norm_write(const float* proj, int ld, const float* conv, int taps, floa
     MapWriteParams p{proj, ld, conv, taps, state, cu_q, token_req, state_slot, qn, kn, eps, slots, q_out, k_cache, v_cache,
                      T, H, G, d, dv, D, page_size, total_pages, (int)run, error_flag_ptr()};
     const dim3 grid((unsigned)((T + run - 1) / run), gy);
-    const bool pairs = d % 2 == 0 && dv % 2 == 0 && D % 4 == 0 && ld % 2 == 0 && aligned16(proj) && aligned16(conv) &&
-                       aligned16(state) && aligned16(qn) && aligned16(kn) && aligned16(q_out) && aligned16(k_cache) &&
-                       aligned16(v_cache);
+    const bool pairs = d % 2 == 0 && dv % 2 == 0 && D % 4 == 0 && ld % 2 == 0 && aligned8(proj) && aligned8(conv) &&
+                       aligned8(state) && aligned8(qn) && aligned8(kn) && aligned8(q_out) && aligned8(k_cache) &&
+                       aligned8(v_cache);
     if (dtype == F32) map_write<float>(p, pairs, grid, stream);
     else map_write<__nv_bfloat16>(p, pairs, grid, stream);
     check_launch("map_norm_write");

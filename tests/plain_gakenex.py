@@ -103,9 +103,11 @@ def weighted_input_experts(h, p, top, rounded=False):
     ids, s = routing(h, p("router"), top)
     hh = as_stored(h, rounded)
     out = torch.zeros_like(h)
-    for t in range(h.shape[0]):
-        for e, w in zip(ids[t].tolist(), s[t]):
-            out[t] += expert(as_stored(w * hh[t], rounded), p, e, rounded)
+    for e in range(p("router").shape[0]):
+        for j in range(top):
+            rows = (ids[:, j] == e).nonzero().flatten()
+            if rows.numel():
+                out[rows] += expert(as_stored(s[rows, j:j + 1] * hh[rows], rounded), p, e, rounded)
     return out
 
 

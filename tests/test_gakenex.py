@@ -473,3 +473,18 @@ def test_a_reader_widens_window_and_kept_start():
                      final_norm=PartSpec("rmsnorm", {"size": 16, "eps": 1e-5}), order=[LayerCall(0), LayerCall(1, reads_cache_of=0)])
     need = DecoderModel(spec, Runtime("cpu", torch.float32, None)).cache_needs()[0][0]
     assert (need.window, need.keep_first) == (9, 7)
+
+
+def test_the_benchmarks_configurations_resolve():
+    """The benchmark's model of this design and the one beside it: equal width, layers, feed-forwards, heads and window."""
+    sys.path.insert(0, os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
+    import bench
+    from dlm_b200.registry import resolve
+    z = bench.gakenex_config(1024)
+    _, cfg, spec = resolve(copy.deepcopy(z))
+    _, q, qspec = resolve(bench.qwen_config_like_gakenex(z))
+    assert len(spec.layers) == len(qspec.layers) == 4 and spec.hidden_size == qspec.hidden_size == 1024
+    att = cfg.layers[0]["mixer"]
+    assert (q.num_attention_heads, q.num_key_value_heads, q.head_dim) == (att["heads"], att["kv_heads"], att["vdim"])
+    assert [L.params["ffn"].kind for L in spec.layers] == ["clamped_glu_dense", "moe_topk"] * 2
+    assert [L.params["ffn"].kind for L in qspec.layers] == ["swiglu_dense", "moe_softmax_topk"] * 2
