@@ -1600,12 +1600,8 @@ def gakenex_kernels(z, pk, batch, context, prefill_tokens):
             ids = torch.randint(0, V, (T,), **i32)
             emb, pos = (torch.randn(V, W, device=dev).to(bf), torch.randn(8192, W, device=dev).to(bf))
             nw = torch.randn(W, device=dev)
-
-            def entry():
-                x = ops.embed(ids, emb)
-                ops.add_rows(x, pos, b.positions)
-                return ops.rmsnorm(x, nw, 1e-6, torch.float32)
-            timed("embedding, positions and norm", case, entry, T * W * 8)
+            timed("embed_norm (embedding, positions and norm)", case,
+                  lambda: ops.embed_norm(ids, emb, 1.0, pos, b.positions, nw, 1e-6), T * W * 8)
             timed("embedding (Qwen2's)", case, lambda: ops.embed(ids, emb), T * W * 6)
             # ---- the two-map head: convolution, norms and write; attention; difference, norm and gate
             H, G, d, dv, taps = att["heads"], att["kv_heads"], att["dim"], att["vdim"], att["conv"]

@@ -24,6 +24,11 @@ enum Epilogue : int {
 void embed(const int32_t* tokens, const void* table, float* out, int T, int H, int V, float scale, int dtype,
            cudaStream_t stream);
 
+// out[t] (f32) = v / sqrt(mean(v^2) + eps) * w with v = table[tokens[t], :] * scale + added[idx[t], :] (added == nullptr: no
+// second term); both tables in `dtype`, H at most 51,200.  An id outside its table sets error 1 (tokens) or 6 (idx).
+void embed_norm(const int32_t* tokens, const void* table, const void* added, const int32_t* idx, const float* w, float* out,
+                int T, int H, int V, int n_added, float scale, float eps, int dtype, cudaStream_t stream);
+
 // out[i, :] = x[rows ? rows[i] : i, :] * rsqrt(mean(x^2) + eps) * w      (x, w f32; out dtype given)
 void rmsnorm(const float* x, const float* w, void* out, const int32_t* rows, int n_rows, int H, float eps,
              int out_dtype, cudaStream_t stream);

@@ -26,6 +26,11 @@ PYBIND11_MODULE(_dlm_kernels, m) {
         dlmk::embed(ptr<const int32_t>(tokens), ptr<const void>(table), ptr<float>(out), T, H, V, scale, dtype,
                     st(stream));
     });
+    m.def("embed_norm", [](u64 tokens, u64 table, u64 added, u64 idx, u64 w, u64 out, int T, int H, int V, int n_added,
+                           float scale, float eps, int dtype, u64 stream) {
+        dlmk::embed_norm(ptr<const int32_t>(tokens), ptr<const void>(table), ptr<const void>(added), ptr<const int32_t>(idx),
+                         ptr<const float>(w), ptr<float>(out), T, H, V, n_added, scale, eps, dtype, st(stream));
+    });
     m.def("rmsnorm", [](u64 x, u64 w, u64 out, u64 rows, int n_rows, int H, float eps, int out_dtype, u64 stream) {
         dlmk::rmsnorm(ptr<const float>(x), ptr<const float>(w), ptr<void>(out), ptr<const int32_t>(rows), n_rows, H,
                       eps, out_dtype, st(stream));

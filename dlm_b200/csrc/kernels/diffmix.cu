@@ -5,66 +5,12 @@
 // key/value heads then gives both maps over the same values, which are stored once.
 #include "api.h"
 #include "common.cuh"
+#include "lanes.cuh"
 
 namespace dlmk {
 namespace {
 
 constexpr int HEAD_WARPS = 8;
-
-template <int V> struct Lanes { float v[V]; };
-template <int V> __device__ __forceinline__ Lanes<V> load_f32(const float* p) {
-    Lanes<V> r;
-    if constexpr (V == 4) {
-        const float4 x = *reinterpret_cast<const float4*>(p);
-        r.v[0] = x.x; r.v[1] = x.y; r.v[2] = x.z; r.v[3] = x.w;
-    } else if constexpr (V == 2) {
-        const float2 x = *reinterpret_cast<const float2*>(p);
-        r.v[0] = x.x; r.v[1] = x.y;
-    } else {
-        r.v[0] = *p;
-    }
-    return r;
-}
-template <int V> __device__ __forceinline__ Lanes<V> load_act(const float* p) { return load_f32<V>(p); }
-template <int V> __device__ __forceinline__ Lanes<V> load_act(const __nv_bfloat16* p) {
-    Lanes<V> r;
-    if constexpr (V == 1) {
-        r.v[0] = __bfloat162float(*p);
-    } else {
-        uint32_t w[V / 2];
-        if constexpr (V == 4) {
-            const uint2 x = *reinterpret_cast<const uint2*>(p);
-            w[0] = x.x; w[1] = x.y;
-        } else {
-            w[0] = *reinterpret_cast<const uint32_t*>(p);
-        }
-#pragma unroll
-        for (int i = 0; i < V / 2; ++i) {
-            r.v[2 * i] = __uint_as_float(w[i] << 16);
-            r.v[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
-        }
-    }
-    return r;
-}
-template <int V> __device__ __forceinline__ void store_act(float* p, const Lanes<V>& r) {
-    if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(r.v[0], r.v[1], r.v[2], r.v[3]);
-    else if constexpr (V == 2) *reinterpret_cast<float2*>(p) = make_float2(r.v[0], r.v[1]);
-    else *p = r.v[0];
-}
-template <int V> __device__ __forceinline__ void store_act(__nv_bfloat16* p, const Lanes<V>& r) {
-    if constexpr (V == 1) {
-        *p = __float2bfloat16_rn(r.v[0]);
-    } else {
-        uint32_t w[V / 2];
-#pragma unroll
-        for (int i = 0; i < V / 2; ++i) {
-            const __nv_bfloat162 b = __floats2bfloat162_rn(r.v[2 * i], r.v[2 * i + 1]);
-            w[i] = *reinterpret_cast<const uint32_t*>(&b);
-        }
-        if constexpr (V == 4) *reinterpret_cast<uint2*>(p) = make_uint2(w[0], w[1]);
-        else *reinterpret_cast<uint32_t*>(p) = w[0];
-    }
-}
 
 struct MapWriteParams {
     const float* proj; int ld;          // rows [q: H x 2 x d | k: G x 2 x d | v: G x dv | ...]
@@ -74,114 +20,154 @@ struct MapWriteParams {
     const float* qn; const float* kn; float eps;
     const int32_t* slots;
     void* q_out; void* k_cache; void* v_cache;
-    int T, H, G, d, dv, D, page_size, total_pages, run;
+    int T, H, G, d, dv, D, page_size, page_shift, total_pages;
     int* err;
 };
 
-// A warp takes one map of one query or key head, or one value head, and `run` tokens: the convolution over time, the
-// norm over the map's d entries (not for values), the query into its half of q_out, key and value into the token's slot.
+// A warp takes one query or key head (both maps, side by side in the rows) or one value head, and RUN tokens: the
+// convolution over time, a norm over each map's d entries (not for values), the two queries into their halves of q_out,
+// key and value into the token's slot.  The rows of all its tokens (and of the taps - 1 before them) are asked for at once.
 // Where a request brings a single token the warp also moves the carried inputs of its channels on: nobody else reads
-// them in this launch.  NP groups of V neighbouring entries a lane; TAPS 0: any number of taps.
-template <typename T, int V, int NP, int TAPS>
+// them in this launch.  NP groups of V neighbouring entries a lane (V divides d and dv, so that a group lies in one map);
+// TAPS taps (1: no convolution over several tokens), 0: any number (read from the parameters, the rows then one by one).
+template <typename T, int V, int NP, int TAPS, int RUN>
 __global__ void __launch_bounds__(HEAD_WARPS * 32) map_norm_write_kernel(MapWriteParams p) {
     dep_wait();
     dep_launch_next();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int item = blockIdx.y * HEAD_WARPS + warp;
-    const int nq = 2 * p.H, nk = 2 * p.G;
-    if (item >= nq + nk + p.G) return;
-    const bool is_q = item < nq, is_v = item >= nq + nk;
-    const int width = is_v ? p.dv : p.d;
-    const int c0 = is_v ? (nq + nk) * p.d + (item - nq - nk) * p.dv : item * p.d;
-    const int C = (nq + nk) * p.d + p.G * p.dv;
-    const int taps = p.conv == nullptr ? 1 : (TAPS > 0 ? TAPS : p.taps);
-    const int keep = taps - 1;
-    const int half = p.D / 2;
-    const float* norm = is_q ? p.qn : p.kn;
-    T* q_out = static_cast<T*>(p.q_out);
-    T* kv = static_cast<T*>(is_v ? p.v_cache : p.k_cache);
-    const int t_end = min(p.T, ((int)blockIdx.x + 1) * p.run);
-    for (int t = blockIdx.x * p.run; t < t_end; ++t) {
-        const int r = p.token_req[t];
-        const int start = p.cu_q[r], n = p.cu_q[r + 1] - start;
-        float* st = keep > 0 ? p.state + (long long)p.state_slot[r] * keep * C + c0 : nullptr;
-        const float* x = p.proj + (long long)t * p.ld + c0;
+    if (item >= p.H + 2 * p.G) return;
+    const bool is_q = item < p.H, is_v = item >= p.H + p.G;
+    const int d = p.d, half = p.D / 2;
+    const int width = is_v ? p.dv : 2 * d;
+    const int c0 = is_v ? 2 * (p.H + p.G) * d + (item - p.H - p.G) * p.dv : item * 2 * d;
+    const int C = 2 * (p.H + p.G) * d + p.G * p.dv;
+    const int keep = (TAPS > 0 ? TAPS : p.taps) - 1;
+    const float* conv = p.conv != nullptr ? p.conv + c0 : nullptr;
+    const int t0 = blockIdx.x * RUN;
+    const float* x0 = p.proj + (long long)t0 * p.ld + c0;               // the run's first row
+    constexpr int LEAD = TAPS > 0 ? TAPS - 1 : 0;                       // rows in front of the run
+    constexpr int ROWS = RUN + LEAD;
+    Lanes<V> rows[ROWS][NP], w[TAPS > 0 ? TAPS : 1][NP], nw[NP];
+#pragma unroll
+    for (int i = 0; i < NP; ++i) {
+        const int e = (i * 32 + lane) * V;
+        const bool on = e < width;
+#pragma unroll
+        for (int a = 0; a < ROWS; ++a) {
+            const int t = t0 + a - LEAD;
+            if (on && t >= 0 && t < p.T) rows[a][i] = load_f32<V>(x0 + (a - LEAD) * p.ld + e);
+        }
+        if (on && TAPS > 0 && conv != nullptr) {
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) w[j][i] = load_f32<V>(conv + j * C + e);
+        }
+        if (on && !is_v) nw[i] = load_f32<V>((is_q ? p.qn : p.kn) + (e < d ? e : e - d));
+    }
+    // the request of the run's first token; most runs lie in one request
+    int r = p.token_req[t0], start = p.cu_q[r], count = p.cu_q[r + 1] - start;
+    float* st = p.state + (long long)p.state_slot[r] * keep * C + c0;
+    const int t_end = min(p.T, t0 + RUN);
+    const bool same = p.token_req[t_end - 1] == r;
+    const bool inside = same && t0 - keep >= start;                     // nobody needs a carried input
+    Lanes<V> zero;
+#pragma unroll
+    for (int u = 0; u < V; ++u) zero.v[u] = 0.f;
+#pragma unroll
+    for (int a = 0; a < RUN; ++a) {
+        const int t = t0 + a;
+        if (t >= p.T) break;
+        if (!same) {
+            r = p.token_req[t];
+            start = p.cu_q[r];
+            count = p.cu_q[r + 1] - start;
+            st = p.state + (long long)p.state_slot[r] * keep * C + c0;
+        }
         Lanes<V> y[NP];
-        float ss = 0.f;
 #pragma unroll
         for (int i = 0; i < NP; ++i) {
             const int e = (i * 32 + lane) * V;
+            y[i] = zero;
+            if (e >= width) continue;
+            if (conv == nullptr) {
+                y[i] = rows[a + LEAD][i];
+            } else if constexpr (TAPS > 0) {
 #pragma unroll
-            for (int u = 0; u < V; ++u) y[i].v[u] = 0.f;
-            if (e < width) {
-                if (p.conv == nullptr) {
-                    y[i] = load_f32<V>(x + e);
-                } else {
-                    auto add = [&](int j) {
-                        const int back = keep - j;               // how many tokens before t
-                        const Lanes<V> u = t - back >= start ? load_f32<V>(x - (long long)back * p.ld + e)
-                                                             : load_f32<V>(st + (long long)(keep + (t - back - start)) * C + e);
-                        const Lanes<V> w = load_f32<V>(p.conv + (long long)j * C + c0 + e);
+                for (int j = 0; j < TAPS; ++j) {
+                    Lanes<V> u = rows[a + j][i];                        // TAPS - 1 - j tokens before t
+                    if (!inside && t - (TAPS - 1 - j) < start) u = load_f32<V>(st + (j + t - start) * C + e);
 #pragma unroll
-                        for (int k = 0; k < V; ++k) y[i].v[k] = fmaf(w.v[k], u.v[k], y[i].v[k]);
-                    };
-                    if constexpr (TAPS > 0) {
-#pragma unroll
-                        for (int j = 0; j < TAPS; ++j) add(j);
-                    } else {
-                        for (int j = 0; j < taps; ++j) add(j);
-                    }
-                    if (n == 1 && keep > 0) {
-                        for (int j = 0; j + 1 < keep; ++j) store_act<V>(st + (long long)j * C + e, load_f32<V>(st + (long long)(j + 1) * C + e));
-                        store_act<V>(st + (long long)(keep - 1) * C + e, load_f32<V>(x + e));
-                    }
+                    for (int k = 0; k < V; ++k) y[i].v[k] = fmaf(w[j][i].v[k], u.v[k], y[i].v[k]);
                 }
+            } else {
+                for (int j = 0; j <= keep; ++j) {
+                    const int back = keep - j;
+                    const Lanes<V> u = t - back >= start ? load_f32<V>(x0 + (a - back) * p.ld + e)
+                                                         : load_f32<V>(st + (j + t - start) * C + e);
+                    const Lanes<V> wj = load_f32<V>(conv + j * C + e);
 #pragma unroll
-                for (int u = 0; u < V; ++u) ss = fmaf(y[i].v[u], y[i].v[u], ss);
+                    for (int k = 0; k < V; ++k) y[i].v[k] = fmaf(wj.v[k], u.v[k], y[i].v[k]);
+                }
+            }
+            if (conv != nullptr && count == 1 && keep > 0) {
+                for (int j = 0; j + 1 < keep; ++j) store_act<V>(st + j * C + e, load_f32<V>(st + (j + 1) * C + e));
+                store_act<V>(st + (keep - 1) * C + e, rows[a + LEAD][i]);
             }
         }
-        int slot = -1;
-        if (!is_q) {
-            slot = p.slots[t];
+        T* dst;
+        if (is_q) {
+            dst = static_cast<T*>(p.q_out) + ((long long)t * p.H + item) * 2 * p.D;
+        } else {
+            int slot = p.slots[t];
             if (slot >= p.total_pages * p.page_size) {
                 if (lane == 0) *p.err = 2;
                 slot = -1;
             }
             if (slot < 0) continue;
+            const int page = p.page_shift >= 0 ? slot >> p.page_shift : slot / p.page_size;
+            const int g = is_v ? item - p.H - p.G : item - p.H;
+            dst = static_cast<T*>(is_v ? p.v_cache : p.k_cache) +
+                  (((long long)page * p.G + g) * p.page_size + (slot - page * p.page_size)) * p.D;
         }
-        if (!is_v) {
-            ss = warp_sum(ss);
-            const float inv = 1.0f / sqrtf(ss / (float)p.d + p.eps);
+        if (is_v) {
 #pragma unroll
             for (int i = 0; i < NP; ++i) {
                 const int e = (i * 32 + lane) * V;
-                if (e < width) {
-                    const Lanes<V> w = load_f32<V>(norm + e);
-#pragma unroll
-                    for (int u = 0; u < V; ++u) y[i].v[u] = (y[i].v[u] * inv) * w.v[u];
-                }
+                if (e < width) store_act<V>(dst + e, y[i]);
             }
+            for (int e = p.dv + lane; e < p.D; e += 32) dst[e] = from_f32<T>(0.f);
+            continue;
         }
-        // a map fills its half of the stored head, a value head all of it; entries beyond the own size are zeros
-        const int span = is_v ? p.D : half;
-        T* dst;
-        if (is_q) {
-            dst = q_out + ((long long)t * nq + item) * p.D;
-        } else {
-            const int g = is_v ? item - nq - nk : (item - nq) >> 1;
-            dst = kv + (((long long)(slot / p.page_size) * p.G + g) * p.page_size + slot % p.page_size) * p.D;
-        }
-        const int at = is_v ? 0 : (item & 1) * half;                    // nq is even: the map's number for keys as well
-        Lanes<V> zero;
+        float ss0 = 0.f, ss1 = 0.f;
 #pragma unroll
-        for (int u = 0; u < V; ++u) zero.v[u] = 0.f;
+        for (int i = 0; i < NP; ++i) {
+            float q = 0.f;
+#pragma unroll
+            for (int u = 0; u < V; ++u) q = fmaf(y[i].v[u], y[i].v[u], q);
+            if ((i * 32 + lane) * V < d) ss0 += q; else ss1 += q;       // (beyond the head's own entries y is zero)
+        }
+        const float inv0 = 1.0f / sqrtf(warp_sum(ss0) / (float)d + p.eps);
+        const float inv1 = 1.0f / sqrtf(warp_sum(ss1) / (float)d + p.eps);
+        // map 1 goes to [0, d), map 2 to [half, half + d) of a key; of the two queries' rows likewise, with zeros in the
+        // other map's place
 #pragma unroll
         for (int i = 0; i < NP; ++i) {
             const int e = (i * 32 + lane) * V;
-            if (e < span) {
-                store_act<V>(dst + at + e, y[i]);
-                if (is_q) store_act<V>(dst + (half - at) + e, zero);
+            if (e >= width) continue;
+            const bool second = e >= d;
+            const int at = second ? half + e - d : e;
+#pragma unroll
+            for (int u = 0; u < V; ++u) y[i].v[u] = (y[i].v[u] * (second ? inv1 : inv0)) * nw[i].v[u];
+            if (is_q) {
+                store_act<V>(dst + (second ? p.D : 0) + at, y[i]);
+                store_act<V>(dst + (second ? 0 : p.D) + at, zero);
+            } else {
+                store_act<V>(dst + at, y[i]);
             }
+        }
+        for (int e = d + lane; e < half; e += 32) {                     // where a half is wider than a map
+            dst[e] = dst[half + e] = from_f32<T>(0.f);
+            if (is_q) dst[p.D + e] = dst[p.D + half + e] = from_f32<T>(0.f);
         }
     }
 }
@@ -250,24 +236,33 @@ __global__ void weigh_rows_kernel(const T* h, const float* wts, const int32_t* d
     }
 }
 
-template <typename T, int V, int NP>
-void launch_map_write(const MapWriteParams& p, dim3 grid, cudaStream_t stream) {
-    const dim3 block(HEAD_WARPS * 32);
-    if (p.conv != nullptr && p.taps == 3) launch_dep(map_norm_write_kernel<T, V, NP, 3>, grid, block, 0, stream, p);
-    else if (p.conv != nullptr && p.taps == 4) launch_dep(map_norm_write_kernel<T, V, NP, 4>, grid, block, 0, stream, p);
-    else launch_dep(map_norm_write_kernel<T, V, NP, 0>, grid, block, 0, stream, p);
+template <typename T, int V, int NP, int RUN>
+void launch_map_write(const MapWriteParams& p, int gy, cudaStream_t stream) {
+    const dim3 grid((p.T + RUN - 1) / RUN, gy), block(HEAD_WARPS * 32);
+    if (p.taps == 1) launch_dep(map_norm_write_kernel<T, V, NP, 1, RUN>, grid, block, 0, stream, p);
+    else if (p.taps == 3) launch_dep(map_norm_write_kernel<T, V, NP, 3, RUN>, grid, block, 0, stream, p);
+    else if (p.taps == 4) launch_dep(map_norm_write_kernel<T, V, NP, 4, RUN>, grid, block, 0, stream, p);
+    else launch_dep(map_norm_write_kernel<T, V, NP, 0, RUN>, grid, block, 0, stream, p);
 }
 
 template <typename T>
-void map_write(const MapWriteParams& p, bool pairs, dim3 grid, cudaStream_t stream) {
-    if (pairs) {
-        if (p.D <= 64) launch_map_write<T, 2, 1>(p, grid, stream);
-        else if (p.D <= 128) launch_map_write<T, 2, 2>(p, grid, stream);
-        else launch_map_write<T, 2, 4>(p, grid, stream);
+void map_write(const MapWriteParams& p, int vec, int gy, cudaStream_t stream) {
+    // a token a warp until the machine is full several times over, then four
+    const bool many = (long long)p.T * gy > 16LL * sm_count();
+#define DLM_MAP(V, NP)                                                                                                 \
+    do { if (many) launch_map_write<T, V, NP, 4>(p, gy, stream); else launch_map_write<T, V, NP, 1>(p, gy, stream); } while (0)
+    if (vec == 4) {
+        if (p.D <= 128) DLM_MAP(4, 1);
+        else DLM_MAP(4, 2);
+    } else if (vec == 2) {
+        if (p.D <= 64) DLM_MAP(2, 1);
+        else if (p.D <= 128) DLM_MAP(2, 2);
+        else DLM_MAP(2, 4);
     } else {
-        if (p.D <= 128) launch_map_write<T, 1, 4>(p, grid, stream);
-        else launch_map_write<T, 1, 8>(p, grid, stream);
+        if (p.D <= 128) DLM_MAP(1, 4);
+        else DLM_MAP(1, 8);
     }
+#undef DLM_MAP
 }
 
 template <typename T>
@@ -283,7 +278,6 @@ void diff_norm_gate_of(const void* o, const float* gate, int ldg, void* out, lon
 }
 
 bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
-bool aligned8(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 7) == 0; }
 
 }  // namespace
 
@@ -295,18 +289,21 @@ void map_norm_write(const float* proj, int ld, const float* conv, int taps, floa
     DLM_CHECK(D % 2 == 0 && D <= 256 && 2 * d <= D && dv <= D, "map_norm_write: a stored head (at most 256 wide) holds two keys or a value");
     DLM_CHECK(conv == nullptr || (taps >= 1 && taps <= 16), "map_norm_write: 1 to 16 taps");
     DLM_CHECK(conv == nullptr || taps == 1 || state != nullptr, "map_norm_write: a convolution over several tokens carries its inputs");
-    const int items = 2 * H + 3 * G, gy = (items + HEAD_WARPS - 1) / HEAD_WARPS;
-    // a token a warp until the machine is full several times over, then runs of tokens (they share the convolution's rows)
-    long long run = (long long)T * gy / (8LL * sm_count());
-    run = run < 1 ? 1 : (run > 8 ? 8 : run);
-    MapWriteParams p{proj, ld, conv, taps, state, cu_q, token_req, state_slot, qn, kn, eps, slots, q_out, k_cache, v_cache,
-                     T, H, G, d, dv, D, page_size, total_pages, (int)run, error_flag_ptr()};
-    const dim3 grid((unsigned)((T + run - 1) / run), gy);
-    const bool pairs = d % 2 == 0 && dv % 2 == 0 && D % 4 == 0 && ld % 2 == 0 && aligned8(proj) && aligned8(conv) &&
-                       aligned8(state) && aligned8(qn) && aligned8(kn) && aligned8(q_out) && aligned8(k_cache) &&
-                       aligned8(v_cache);
-    if (dtype == F32) map_write<float>(p, pairs, grid, stream);
-    else map_write<__nv_bfloat16>(p, pairs, grid, stream);
+    const int gy = (H + 2 * G + HEAD_WARPS - 1) / HEAD_WARPS;
+    MapWriteParams p{proj, ld, conv, conv != nullptr ? taps : 1, state, cu_q, token_req, state_slot, qn, kn, eps, slots,
+                     q_out, k_cache, v_cache, T, H, G, d, dv, D, page_size, -1, total_pages, error_flag_ptr()};
+    if ((page_size & (page_size - 1)) == 0)
+        for (p.page_shift = 0; (1 << p.page_shift) < page_size;) ++p.page_shift;
+    // entries a lane takes side by side: as many as divide the sizes and the addresses allow
+    auto fits = [&](int v) {
+        const uintptr_t f32 = reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(conv) |
+                              reinterpret_cast<uintptr_t>(state) | reinterpret_cast<uintptr_t>(qn) | reinterpret_cast<uintptr_t>(kn);
+        const uintptr_t act = reinterpret_cast<uintptr_t>(q_out) | reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache);
+        return d % v == 0 && dv % v == 0 && D % (2 * v) == 0 && ld % v == 0 && f32 % (4 * v) == 0 && act % (4 * v) == 0;
+    };
+    const int vec = fits(4) ? 4 : (fits(2) ? 2 : 1);
+    if (dtype == F32) map_write<float>(p, vec, gy, stream);
+    else map_write<__nv_bfloat16>(p, vec, gy, stream);
     check_launch("map_norm_write");
     if (conv != nullptr && taps > 1 && num_single < R)
         conv_state(proj, ld, state, cu_q, state_slot, R, 2 * (H + G) * d + G * dv, taps, 1, stream);

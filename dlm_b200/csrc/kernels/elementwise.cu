@@ -4,6 +4,7 @@
 #include <cstdlib>
 
 #include "common.cuh"
+#include "lanes.cuh"
 
 namespace dlmk {
 
@@ -72,6 +73,52 @@ __global__ void embed_kernel(const int32_t* __restrict__ tokens, const T* __rest
     }
     const T* row = table + (long long)tok * H;
     for (int i = threadIdx.x; i < H; i += blockDim.x) o[i] = to_f32(row[i]) * scale;
+}
+
+// out[t] = rmsnorm(table[tokens[t]] * scale + added[idx[t]]) * w (added == nullptr: only the tokens): what the first layer
+// of a model gets that adds a vector per position and norms the sum.  A block a token; the row stays in shared memory.
+template <typename T, int V>
+__global__ void embed_norm_kernel(const int32_t* __restrict__ tokens, const T* __restrict__ table, const T* __restrict__ added,
+                                  const int32_t* __restrict__ idx, const float* __restrict__ w, float* out, int H, int vocab,
+                                  int n_added, float scale, float eps, int* err) {
+    extern __shared__ __align__(16) float embed_row[];
+    __shared__ float s_part[32];
+    dep_wait();
+    dep_launch_next();
+    const int t = blockIdx.x;
+    const int tok = tokens[t], at = added != nullptr ? idx[t] : 0;
+    float* o = out + (long long)t * H;
+    const bool bad_tok = tok < 0 || tok >= vocab, bad_at = added != nullptr && (at < 0 || at >= n_added);
+    if (bad_tok || bad_at) {       // never read outside a table
+        if (threadIdx.x == 0) *err = bad_tok ? 1 : 6;
+        for (int i = threadIdx.x; i < H; i += blockDim.x) o[i] = 0.f;
+        return;
+    }
+    const T* row = table + (long long)tok * H;
+    const T* more = added != nullptr ? added + (long long)at * H : nullptr;
+    float ss = 0.f;
+    for (int i = threadIdx.x * V; i < H; i += blockDim.x * V) {
+        Lanes<V> x = load_act<V>(row + i);
+        if (more != nullptr) {
+            const Lanes<V> y = load_act<V>(more + i);
+#pragma unroll
+            for (int u = 0; u < V; ++u) x.v[u] = fmaf(x.v[u], scale, y.v[u]);
+        } else {
+#pragma unroll
+            for (int u = 0; u < V; ++u) x.v[u] *= scale;
+        }
+#pragma unroll
+        for (int u = 0; u < V; ++u) ss = fmaf(x.v[u], x.v[u], ss);
+        store_act<V>(embed_row + i, x);
+    }
+    const float inv = 1.0f / sqrtf(block_sum(ss, s_part) / (float)H + eps);
+    for (int i = threadIdx.x * V; i < H; i += blockDim.x * V) {      // a thread rereads what it wrote
+        Lanes<V> x = load_f32<V>(embed_row + i);
+        const Lanes<V> g = load_f32<V>(w + i);
+#pragma unroll
+        for (int u = 0; u < V; ++u) x.v[u] = (x.v[u] * inv) * g.v[u];
+        store_act<V>(o + i, x);
+    }
 }
 
 // ---------------------------------------------------------------------- rmsnorm
@@ -402,6 +449,29 @@ void embed(const int32_t* tokens, const void* table, float* out, int T, int H, i
     if (dtype == F32) launch_dep(embed_kernel<float>, T, threads, 0, stream, tokens, static_cast<const float*>(table), out, H, V, scale, err);
     else launch_dep(embed_kernel<__nv_bfloat16>, T, threads, 0, stream, tokens, static_cast<const __nv_bfloat16*>(table), out, H, V, scale, err);
     check_launch("embed");
+}
+
+void embed_norm(const int32_t* tokens, const void* table, const void* added, const int32_t* idx, const float* w, float* out,
+                int T, int H, int V, int n_added, float scale, float eps, int dtype, cudaStream_t stream) {
+    if (T <= 0) return;
+    const size_t smem = (size_t)H * sizeof(float);
+    DLM_CHECK(smem <= 200 * 1024, "embed_norm: a row does not fit in shared memory");
+    DLM_CHECK(added == nullptr || idx != nullptr, "embed_norm: added rows need their numbers");
+    const bool vec = H % 4 == 0 && ((reinterpret_cast<uintptr_t>(table) | reinterpret_cast<uintptr_t>(added) |
+                                     reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+    const dim3 block(H >= 1024 ? 256 : 128);
+    int* err = error_flag_ptr();
+#define DLM_EN(T_, V_)                                                                                                 \
+    do {                                                                                                              \
+        if (smem > 40 * 1024)                                                                                         \
+            cudaFuncSetAttribute(embed_norm_kernel<T_, V_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);   \
+        launch_dep(embed_norm_kernel<T_, V_>, dim3(T), block, smem, stream, tokens, static_cast<const T_*>(table),    \
+                   static_cast<const T_*>(added), idx, w, out, H, V, n_added, scale, eps, err);                       \
+    } while (0)
+    if (dtype == F32) { if (vec) DLM_EN(float, 4); else DLM_EN(float, 1); }
+    else { if (vec) DLM_EN(__nv_bfloat16, 4); else DLM_EN(__nv_bfloat16, 1); }
+#undef DLM_EN
+    check_launch("embed_norm");
 }
 
 void rmsnorm(const float* x, const float* w, void* out, const int32_t* rows, int n_rows, int H, float eps,

@@ -128,6 +128,22 @@ class NativeOps:
         self.k.embed(_p(tokens), _p(table), _p(out), T, H, V, float(scale), _dt(table.dtype), self._stream())
         return out
 
+    def embed_norm(self, tokens, table, scale, added, idx, w, eps):
+        """``v / sqrt(mean(v^2) + eps) * w`` in 32-bit with ``v = table[tokens] * scale + added[idx]`` (``added`` None: no
+        second term): embedding, a vector per position and their norm in one pass."""
+        T, (V, H) = tokens.numel(), table.shape
+        assert added is None or (added.shape[1] == H and added.dtype == table.dtype)
+        if 4 * H > 200 * 1024:                       # a row too long for the kernel's shared memory
+            x = self.embed(tokens, table, scale)
+            if added is not None:
+                self.add_rows(x, added, idx)
+            return self.rmsnorm(x, w, eps, torch.float32)
+        out = torch.empty((T, H), dtype=torch.float32, device=table.device)
+        self.launches += 1
+        self.k.embed_norm(_p(tokens), _p(table), _p(added), _p(idx), _p(w), _p(out), T, H, V,
+                          0 if added is None else added.shape[0], float(scale), float(eps), _dt(table.dtype), self._stream())
+        return out
+
     def add_rows(self, x, table, idx):
         """``x[t] += table[idx[t]]`` in place (x 32-bit): learned position vectors."""
         T, H = x.shape

@@ -171,6 +171,11 @@ class PositionEncoding(Part):
     def on_embed(self, x: torch.Tensor, positions: torch.Tensor, rt: Runtime) -> None:
         """Hook for encodings that act on the embedded tokens (in place); default: nothing."""
 
+    def added_rows(self):
+        """The table of an encoding that does no more than add row ``position`` of it to the embedded token (a kernel may
+        then do that itself), else None."""
+        return None
+
 
 class Mixer(Part):
     def cache_need(self) -> PagedCache | None:

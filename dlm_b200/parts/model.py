@@ -194,11 +194,16 @@ class DecoderModel:
 
         ctx = StepContext(rt, batch, paged, cache.state_tensor)
         s = self.spec
-        x = ops.embed(batch.tokens, self.embed, s.embed_scale) if s.embed_scale != 1.0 else ops.embed(batch.tokens, self.embed)
-        if self.embed_position is not None:
-            self.embed_position.on_embed(x, batch.positions, rt)
-        if self.embed_norm is not None:
-            x = self.embed_norm.forward(x, rt, out_dtype=torch.float32)
+        rms = self.embed_norm.fusable_rms() if self.embed_norm is not None else None
+        added = self.embed_position.added_rows() if self.embed_position is not None else None
+        if rms is not None and (self.embed_position is None or added is not None):
+            x = ops.embed_norm(batch.tokens, self.embed, s.embed_scale, added, batch.positions, *rms)
+        else:
+            x = ops.embed(batch.tokens, self.embed, s.embed_scale) if s.embed_scale != 1.0 else ops.embed(batch.tokens, self.embed)
+            if self.embed_position is not None:
+                self.embed_position.on_embed(x, batch.positions, rt)
+            if self.embed_norm is not None:
+                x = self.embed_norm.forward(x, rt, out_dtype=torch.float32)
         if s.residual_streams is not None:
             x = ops.streams_expand(x, s.residual_streams)
         # a model with repeated passes keeps the embedded tokens: blocks change x in place

@@ -136,6 +136,9 @@ class LearnedPositions(PositionEncoding):
     def on_embed(self, x, positions, rt: Runtime) -> None:
         rt.ops.add_rows(x, self.table, positions)
 
+    def added_rows(self):
+        return self.table
+
 
 register_part("position", "learned", LearnedPositions)
 register_part("position", "rope_neox", RotaryNeoX)

@@ -38,6 +38,12 @@ class PlainOps:
     def embed(self, tokens, table, scale=1.0):
         return _f(table[tokens.long()]) * scale
 
+    def embed_norm(self, tokens, table, scale, added, idx, w, eps):
+        x = self.embed(tokens, table, scale)
+        if added is not None:
+            self.add_rows(x, added, idx)
+        return self.rmsnorm(x, w, eps, torch.float32)
+
     def add_rows(self, x, table, idx):
         x += _f(table[idx.long()])
 

@@ -172,6 +172,7 @@ def test_a_missing_kept_page_is_reported(ops):
         table[0, 0] = -1
         q = randn(q_len, 128, seed=4, dtype=torch.bfloat16)
         ops.attention(q, k, v, table, cu_q, kv_len, 64, 0.1, 1, 1, 128, q_len, 500, int(q_len == 1), keep_first=10)
+        torch.cuda.synchronize()
         with pytest.raises(Exception, match="no page"):
             ops.check_errors()
 
@@ -250,6 +251,7 @@ def test_convolution_norm_and_write(ops, dtype, H, G, d, dv, D, taps, off):
     bad = slots.clone()
     bad[0] = 21 * ps
     ops.map_norm_write(proj, w, gs if taps > 1 else None, b, qn, kn, 1e-3, bad, kc, vc, H, G, d, dv, D, dtype)
+    torch.cuda.synchronize()              # (the flag is set once the kernel has run)
     with pytest.raises(Exception, match="slot"):
         ops.check_errors()
 
@@ -273,6 +275,28 @@ def test_difference_norm_and_gate(ops, dtype, H, dv, D, off, T):
             want = ref.diff_norm_gate(o.cpu(), None if g is None else g.cpu(), H, dv, D, lam, 1e-4, 0.65)
             assert got.dtype == dtype and torch.allclose(got.float().cpu(), want.float(), **tol(dtype, 2e-5, 1e-2))
     ops.check_errors()
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("T,H", [(1, 192), (40, 63), (300, 2048), (3, 12288), (2, 12292), (1, 51204), (5, 1030)])
+def test_embedding_positions_and_norm(ops, dtype, T, H):
+    """One pass for the token's row, the position's row and their norm; a large eps, a scale, no positions; ids outside
+    their tables are reported and nothing is read."""
+    ref = PlainOps()
+    table, pos = randn(50, H, seed=1, dtype=dtype), randn(33, H, seed=2, std=2.0, dtype=dtype)
+    g = torch.Generator().manual_seed(3)
+    ids, at = (torch.randint(0, n, (T,), generator=g).to(DEV, torch.int32) for n in (50, 33))
+    w = randn(H, seed=4)
+    for scale, added, eps in ((1.0, pos, 0.7), (1.0, None, 1e-6), (3.5, pos, 1e-5)):
+        got = ops.embed_norm(ids, table, scale, added, at, w, eps)
+        want = ref.embed_norm(ids.cpu(), table.cpu(), scale, None if added is None else added.cpu(), at.cpu(), w.cpu(), eps)
+        assert got.dtype == torch.float32 and torch.allclose(got.cpu(), want, atol=1e-5, rtol=1e-5)
+    ops.check_errors()
+    for bad_ids, bad_at, what in ((ids + 50, at, "token id"), (ids, at + 33, "position")):
+        ops.embed_norm(bad_ids, table, 1.0, pos, bad_at, w, 1e-5)
+        torch.cuda.synchronize()
+        with pytest.raises(Exception, match=what):
+            ops.check_errors()
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
