@@ -1621,6 +1621,9 @@ def gakenex_kernels(z, pk, batch, context, prefill_tokens):
             timed("head_norm_rope_write (Salolorn's norm per head, rotation, write)", case,
                   lambda: ops.head_norm_rope_write(hp, b.positions, dn, dn, 1e-6, freq, D, False, slots, k_cache, v_cache, H, G,
                                                    D, D, D, bf), T * (H + 2 * G) * D * 6)
+            timed("rope_kv_write (Qwen2's rotation and write)", case,
+                  lambda: ops.rope_kv_write(hp, b.positions, freq, D, slots, k_cache, v_cache, H, G, D, bf),
+                  T * (H + 2 * G) * D * 6)
             full = torch.zeros(R + 1, taps - 1, C, device=dev)
             conv_wt = conv_w.t().contiguous()
             timed("causal_conv alone (Zesapel's)", case,
