@@ -228,7 +228,6 @@ def test_convolution_norm_and_write(ops, dtype, H, G, d, dv, D, taps, off):
         caches = [torch.full((21, G, ps, D), 7.0, device=DEV, dtype=dtype) for _ in range(2)]
         wk, wv, ws = caches[0].cpu(), caches[1].cpu(), state.cpu()
         kc, vc, gs = caches[0].clone(), caches[1].clone(), state.clone()
-        args = (1e-3,)
         want = ref.map_norm_write(proj.cpu(), None if w is None else w.cpu(), ws, to_cpu(b), qn.cpu(), kn.cpu(), 1e-3, slots.cpu(), wk, wv,
                                   H, G, d, dv, D, dtype)
         got = ops.map_norm_write(proj, w, gs if taps > 1 else None, b, qn, kn, 1e-3, slots, kc, vc, H, G, d, dv, D, dtype)
